@@ -46,7 +46,6 @@ __global__ void __launch_bounds__(192, 1) gemm_persistent_kernel(
   extern __shared__ uint8_t raw[];
   auto& sm = *reinterpret_cast<PersistentStorage<STAGES, FEAT, TC>*>(
       (reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
-  pdl_trigger();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int nkb = (K + TILE_K - 1) / TILE_K;
   const int tiles = m_tiles * n_tiles;
@@ -77,6 +76,7 @@ __global__ void __launch_bounds__(192, 1) gemm_persistent_kernel(
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = sm.tmem_base;
+  pdl_trigger();             // after the allocation, as in the one-tile kernel
 
   if (warp == 0 && lane == 0) {
     // ------------------------------------------------------------------ producer
