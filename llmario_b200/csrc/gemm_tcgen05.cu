@@ -31,7 +31,7 @@
 
 int llm_zero_f32(float* p, int rows, int cols, int ld, cudaStream_t stream);   // elementwise.cu
 int llm_gemm_tcgen05_pair(const void* X, const void* W, void* C, int c_dtype, int T, int N, int K, int lda,
-                          int ldw, int ldc, int mode, int half, int* status, cudaStream_t stream);
+                          int ldw, int ldc, int mode, int half, float limit, int* status, cudaStream_t stream);
 int llm_gemm_tcgen05_persistent(const void* X, const void* W, void* C, int c_dtype, int T, int N, int K,
                                 int lda, int ldw, int ldc, int mode, int half, int* status,
                                 cudaStream_t stream);                        // gemm_tcgen05_persistent.cu
@@ -59,7 +59,9 @@ __global__ void __launch_bounds__(192) gemm_tcgen05_kernel(
     const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
     const __grid_constant__ CUtensorMap map_c, int tma_out, TC* __restrict__ C, int ldc, int T, int N,
     int K, int half, int interleaved, int* __restrict__ status, const int* __restrict__ tile_group,
-    int group_rows, int batch_x_cols, int batch_c_cols) {
+    int group_rows, int batch_x_cols, int batch_c_cols, float limit, const float* __restrict__ row_scale) {
+  // limit, row_scale: of the clamped gated epilogue (row_scale: a factor per row of X on both
+  // products, or null)
   // Batched form (batch_x_cols > 0): blockIdx.z is one of several independent products (a head
   // of a per-head map) instead of a part of K: product z reads the columns z * batch_x_cols .. of
   // X and the matrix z of W (group_rows rows each) and writes the columns z * batch_c_cols .. of C.
@@ -68,9 +70,9 @@ __global__ void __launch_bounds__(192) gemm_tcgen05_kernel(
   extern __shared__ uint8_t raw[];
   auto& sm = *reinterpret_cast<SharedStorage<BN, STAGES>*>(
       (reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
-  pdl_trigger();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int feat_per_tile = EPI == EPI_GATED ? 64 : TILE_M;
+  constexpr bool GATED = gated_epilogue(EPI);
+  const int feat_per_tile = GATED ? 64 : TILE_M;
   const int n0 = blockIdx.x * feat_per_tile;
   const int t0 = blockIdx.y * BN;
   const int kblocks = (K + TILE_K - 1) / TILE_K;
@@ -104,6 +106,9 @@ __global__ void __launch_bounds__(192) gemm_tcgen05_kernel(
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = sm.tmem_base;
+  // only now may the next kernel of the stream be scheduled: every CTA of this one that is
+  // running holds its tensor memory, so a successor that also allocates some cannot starve it
+  pdl_trigger();
   int w_row0 = batched ? (int)blockIdx.z * group_rows : 0;          // first row of this tile's matrix inside W
   bool live = nkb > 0;
   if (tile_group) {
@@ -122,10 +127,10 @@ __global__ void __launch_bounds__(192) gemm_tcgen05_kernel(
         const int s = i % STAGES;
         mbar_expect_tx(&sm.full[s], STAGE_BYTES);
         const int k = (kb_begin + i) * TILE_K;
-        if (EPI == EPI_GATED && interleaved) {
+        if (GATED && interleaved) {
           // the matrix is stored with 16 gate rows, their 16 up rows, the next 16 gate rows, ...
           tma_load_2d(sm.a[s], &map_w, k, w_row0 + 2 * n0, &sm.full[s]);
-        } else if (EPI == EPI_GATED) {
+        } else if (GATED) {
           // 16 gate rows, their 16 up rows, the next 16 gate rows, ...: every 32-lane quarter of
           // the accumulator then holds gate and up of the same 16 features
 #pragma unroll
@@ -190,21 +195,28 @@ __global__ void __launch_bounds__(192) gemm_tcgen05_kernel(
         // With a tensor map for the output the tile is laid out in shared memory as
         // [token][feature] (the pipeline stages are free by now) and written by one TMA store,
         // or added by one TMA reduction (residual add, partial sums of a K split).
-        constexpr int FEAT = EPI == EPI_GATED ? 64 : TILE_M;
+        constexpr int FEAT = GATED ? 64 : TILE_M;
         TC* stage_out = reinterpret_cast<TC*>(&sm.a[0][0]);
 #pragma unroll 1
         for (int c = 0; c < BN; c += 16) {
           uint32_t v[16];
           tmem_ld16(tmem + ((uint32_t)(q * 32) << 16) + (uint32_t)c, v);
           tmem_ld_wait();
-          if (EPI == EPI_GATED) {
+          if (GATED) {
             // lanes 0..15 hold gate of feature q*16 + lane, lanes 16..31 the matching up values
             // (both halves of the warp compute: eight columns each, see gated_columns)
             const int f = q * 16 + (lane & 15);
             const int n = n0 + f;
             const int col0 = c + (lane < 16 ? 0 : 8);
             float r[8];
-            gated_columns<TC>(v, lane, r);
+            if (EPI == EPI_CLAMPED) {
+              float sc[8];
+#pragma unroll
+              for (int i = 0; i < 8; ++i) sc[i] = row_scale ? row_scale[min(t0 + col0 + i, T - 1)] : 1.f;
+              clamped_columns<TC>(v, lane, limit, sc, r);
+            } else {
+              gated_columns<TC>(v, lane, r);
+            }
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
               const int t = t0 + col0 + i;
@@ -388,16 +400,18 @@ namespace {
 template <int BN, int STAGES, int EPI, typename TC>
 int launch(const CUtensorMap& mw, const CUtensorMap& mx, TC* C, int ldc, int T, int N, int K, int half,
            int splits, int interleaved, int* status, cudaStream_t stream, const int* tile_group = nullptr,
-           int group_rows = 0, int batch = 0, int batch_x_cols = 0, int batch_c_cols = 0) {
+           int group_rows = 0, int batch = 0, int batch_x_cols = 0, int batch_c_cols = 0, float act_limit = 0.f,
+           const float* row_scale = nullptr) {
+  constexpr bool GATED = gated_epilogue(EPI);
   // the output goes through TMA when its rows are 16-byte multiples on a 16-byte aligned base
   // (batched: only when a product's columns are whole tiles, since a tile's store is clipped at
   // the matrix's edge alone, and its columns start on a 16-byte boundary)
   CUtensorMap mc = mw;
   int tma_out = 0;
-  const int out_cols = batch ? (batch - 1) * batch_c_cols + N : (EPI == EPI_GATED ? half : N);
+  const int out_cols = batch ? (batch - 1) * batch_c_cols + N : (GATED ? half : N);
   const bool tiles_fit = !batch || (N % TILE_M == 0 && ((size_t)batch_c_cols * sizeof(TC)) % 16 == 0);
   if (tiles_fit && ((uintptr_t)C & 15) == 0 && ((size_t)ldc * sizeof(TC)) % 16 == 0 &&
-      llm_tensor_map(C, T, out_cols, ldc, BN, EPI == EPI_GATED ? 64 : TILE_M, sizeof(TC) == 4 ? 2 : 1, &mc))
+      llm_tensor_map(C, T, out_cols, ldc, BN, GATED ? 64 : TILE_M, sizeof(TC) == 4 ? 2 : 1, &mc))
     tma_out = 1;
   auto kernel = gemm_tcgen05_kernel<BN, STAGES, EPI, TC>;
   constexpr int smem = (int)sizeof(SharedStorage<BN, STAGES>) + 1024;
@@ -407,22 +421,23 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mx, TC* C, int ldc, int T, 
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  const int feat = EPI == EPI_GATED ? 64 : TILE_M;
-  const int limit = EPI == EPI_GATED ? half : N;
+  const int feat = GATED ? 64 : TILE_M;
+  const int limit = GATED ? half : N;
   dim3 grid((limit + feat - 1) / feat, (T + BN - 1) / BN, batch ? batch : splits);
   return launch_pdl(kernel, grid, 192, smem, stream, mw, mx, mc, tma_out, C, ldc, T, N, K, half, interleaved,
-                    status, tile_group, group_rows, batch_x_cols, batch_c_cols);
+                    status, tile_group, group_rows, batch_x_cols, batch_c_cols, act_limit, row_scale);
 }
 
 template <int EPI, typename TC>
 int dispatch(int bn, const CUtensorMap& mw, const CUtensorMap& mx, TC* C, int ldc, int T, int N, int K,
              int half, int splits, int interleaved, int* status, cudaStream_t stream,
-             const int* tile_group = nullptr, int group_rows = 0, int batch = 0, int bx = 0, int bc = 0) {
+             const int* tile_group = nullptr, int group_rows = 0, int batch = 0, int bx = 0, int bc = 0,
+             float limit = 0.f, const float* row_scale = nullptr) {
   switch (bn) {
-    case 16: return launch<16, 6, EPI, TC>(mw, mx, C, ldc, T, N, K, half, splits, interleaved, status, stream, tile_group, group_rows, batch, bx, bc);
-    case 32: return launch<32, 5, EPI, TC>(mw, mx, C, ldc, T, N, K, half, splits, interleaved, status, stream, tile_group, group_rows, batch, bx, bc);
-    case 64: return launch<64, 4, EPI, TC>(mw, mx, C, ldc, T, N, K, half, splits, interleaved, status, stream, tile_group, group_rows, batch, bx, bc);
-    case 128: return launch<128, 3, EPI, TC>(mw, mx, C, ldc, T, N, K, half, splits, interleaved, status, stream, tile_group, group_rows, batch, bx, bc);
+    case 16: return launch<16, 6, EPI, TC>(mw, mx, C, ldc, T, N, K, half, splits, interleaved, status, stream, tile_group, group_rows, batch, bx, bc, limit, row_scale);
+    case 32: return launch<32, 5, EPI, TC>(mw, mx, C, ldc, T, N, K, half, splits, interleaved, status, stream, tile_group, group_rows, batch, bx, bc, limit, row_scale);
+    case 64: return launch<64, 4, EPI, TC>(mw, mx, C, ldc, T, N, K, half, splits, interleaved, status, stream, tile_group, group_rows, batch, bx, bc, limit, row_scale);
+    case 128: return launch<128, 3, EPI, TC>(mw, mx, C, ldc, T, N, K, half, splits, interleaved, status, stream, tile_group, group_rows, batch, bx, bc, limit, row_scale);
   }
   return LLM_ERR_UNSUPPORTED;
 }
@@ -433,12 +448,13 @@ int dispatch(int bn, const CUtensorMap& mw, const CUtensorMap& mx, TC* C, int ld
 //   mode 1: C += X W^T (f32)
 //   mode 2: W = [gate; up] with `half` rows each, C[t][n] = silu(gate) * up, n < half
 //   mode 3: the same with W stored interleaved: 16 gate rows, their 16 up rows, 16 gate rows, ...
+//   mode 4: W as in mode 3, the clamped gated form with `limit` (llm_gemm_tcgen05_clamped)
 // bn: token tile, one of 16, 32, 64, 128, or 256 for the persistent kernel.  out_is_zero: with
 // mode 0 and splits > 1 the caller guarantees that C holds zeros (it is not cleared here).  status: device int, set non-zero when a wait
 // inside the kernel gave up.
-LLM_EXPORT int llm_gemm_tcgen05(const void* X, const void* W, void* C, int c_dtype, int T, int N, int K,
-                                int lda, int ldw, int ldc, int mode, int half, int bn, int splits,
-                                int out_is_zero, int* status, cudaStream_t stream) {
+static int gemm_any(const void* X, const void* W, void* C, int c_dtype, int T, int N, int K,
+                    int lda, int ldw, int ldc, int mode, int half, int bn, int splits,
+                    int out_is_zero, float limit, int* status, cudaStream_t stream) {
   if (T <= 0 || N <= 0) return 0;
   if (K <= 0 || K % 8 || lda % 8 || ldw % 8) return LLM_ERR_UNSUPPORTED;
   if (((uintptr_t)X | (uintptr_t)W) & 15) return LLM_ERR_UNSUPPORTED;
@@ -450,10 +466,10 @@ LLM_EXPORT int llm_gemm_tcgen05(const void* X, const void* W, void* C, int c_dty
     // (the pair kernel cuts K itself where its adding epilogue allows, so it also takes the
     // products for which the caller asked for a split)
     if (splits == 1 || mode == 1) {
-      int r = llm_gemm_tcgen05_pair(X, W, C, c_dtype, T, N, K, lda, ldw, ldc, mode, half, status, stream);
+      int r = llm_gemm_tcgen05_pair(X, W, C, c_dtype, T, N, K, lda, ldw, ldc, mode, half, limit, status, stream);
       if (r != LLM_ERR_UNSUPPORTED) return r;
     }
-    if (splits == 1) {
+    if (splits == 1 && mode != 4) {
       int r = llm_gemm_tcgen05_persistent(X, W, C, c_dtype, T, N, K, lda, ldw, ldc, mode, half, status, stream);
       if (r != LLM_ERR_UNSUPPORTED) return r;
     }
@@ -489,22 +505,47 @@ LLM_EXPORT int llm_gemm_tcgen05(const void* X, const void* W, void* C, int c_dty
       return dispatch<EPI_GATED, float>(bn, mw, mx, (float*)C, ldc, T, N, K, half, 1, mode == 3, status, stream);
     return LLM_ERR_UNSUPPORTED;
   }
+  if (mode == 4) {
+    if (N != 2 * half || half % 16) return LLM_ERR_ARGUMENT;
+    if (c_dtype == LLM_BF16)
+      return dispatch<EPI_CLAMPED, bf16>(bn, mw, mx, (bf16*)C, ldc, T, N, K, half, 1, 1, status, stream, nullptr, 0, 0,
+                                         0, 0, limit);
+    return LLM_ERR_UNSUPPORTED;
+  }
   return LLM_ERR_ARGUMENT;
+}
+
+LLM_EXPORT int llm_gemm_tcgen05(const void* X, const void* W, void* C, int c_dtype, int T, int N, int K,
+                                int lda, int ldw, int ldc, int mode, int half, int bn, int splits,
+                                int out_is_zero, int* status, cudaStream_t stream) {
+  if (mode < 0 || mode > 3) return LLM_ERR_ARGUMENT;
+  return gemm_any(X, W, C, c_dtype, T, N, K, lda, ldw, ldc, mode, half, bn, splits, out_is_zero, 0.f, status, stream);
+}
+
+// C [T][half] bfloat16 = g sigmoid(1.702 g) (u + 1), g = min(X W_gate^T, limit), u = clamp(X W_up^T, -limit,
+// limit); W stored as 16 gate rows, their 16 up rows, 16 gate rows, ... (half a multiple of 16)
+LLM_EXPORT int llm_gemm_tcgen05_clamped(const void* X, const void* W, void* C, int T, int half, int K, int lda,
+                                        int ldw, int ldc, int bn, float limit, int* status, cudaStream_t stream) {
+  return gemm_any(X, W, C, LLM_BF16, T, 2 * half, K, lda, ldw, ldc, 4, half, bn, 1, 0, limit, status, stream);
 }
 
 // The grouped product: W holds `groups` matrices [N][K] one below the other; the rows of X come in
 // tiles of `bn` (16, 32, 64 or 128) and tile y is multiplied with matrix tile_group[y] (device
 // int32 [ceil(T / bn)], made by an earlier kernel of the stream; a negative entry leaves the tile
 // out, its output rows are not written).  mode 0: C = X W_g^T (bf16 or f32); mode 2: W_g = [gate;
-// up] of `half` rows each and C = silu(gate) * up.  No split of K.
+// up] of `half` rows each and C = silu(gate) * up; mode 3: the same with the rows of W_g as 16 gate
+// rows, their 16 up rows, ... (one box of weights per block of K instead of eight); mode 4: W_g as in
+// mode 3, the clamped gated form with `limit`, row_scale [T] (or null) a factor per row of X on both
+// products (C bf16).  No split of K.
 LLM_EXPORT int llm_gemm_tcgen05_grouped(const void* X, const void* W, void* C, int c_dtype, int T, int N, int K,
                                         int lda, int ldw, int ldc, int mode, int half, int bn, int groups,
-                                        const int* tile_group, int* status, cudaStream_t stream) {
+                                        const int* tile_group, float limit, const float* row_scale, int* status,
+                                        cudaStream_t stream) {
   if (T <= 0 || N <= 0 || groups <= 0) return 0;
   if (K <= 0 || K % 8 || lda % 8 || ldw % 8) return LLM_ERR_UNSUPPORTED;
   if (((uintptr_t)X | (uintptr_t)W) & 15) return LLM_ERR_UNSUPPORTED;
-  if (!tile_group || (mode != 0 && mode != 2)) return LLM_ERR_ARGUMENT;
-  if (mode == 2 && (N != 2 * half || half % 16)) return LLM_ERR_UNSUPPORTED;   // (a box of 16 rows stays inside its matrix)
+  if (!tile_group || mode < 0 || mode == 1 || mode > 4) return LLM_ERR_ARGUMENT;
+  if (mode >= 2 && (N != 2 * half || half % 16)) return LLM_ERR_UNSUPPORTED;   // (a box of 16 rows stays inside its matrix)
   if ((long long)groups * N > 0x7fffffffLL) return LLM_ERR_UNSUPPORTED;
   CUtensorMap mw, mx;
   if (!llm_tensor_map(W, (long long)groups * N, K, ldw, mode == 2 ? 16 : TILE_M, TILE_K, 0, &mw))
@@ -517,10 +558,15 @@ LLM_EXPORT int llm_gemm_tcgen05_grouped(const void* X, const void* W, void* C, i
       return dispatch<EPI_STORE, bf16>(bn, mw, mx, (bf16*)C, ldc, T, N, K, half, 1, 0, status, stream, tile_group, N);
     return LLM_ERR_UNSUPPORTED;
   }
+  if (mode == 4) {
+    if (c_dtype != LLM_BF16) return LLM_ERR_UNSUPPORTED;
+    return dispatch<EPI_CLAMPED, bf16>(bn, mw, mx, (bf16*)C, ldc, T, N, K, half, 1, 1, status, stream, tile_group, N, 0,
+                                       0, 0, limit, row_scale);
+  }
   if (c_dtype == LLM_BF16)
-    return dispatch<EPI_GATED, bf16>(bn, mw, mx, (bf16*)C, ldc, T, N, K, half, 1, 0, status, stream, tile_group, N);
+    return dispatch<EPI_GATED, bf16>(bn, mw, mx, (bf16*)C, ldc, T, N, K, half, 1, mode == 3, status, stream, tile_group, N);
   if (c_dtype == LLM_F32)
-    return dispatch<EPI_GATED, float>(bn, mw, mx, (float*)C, ldc, T, N, K, half, 1, 0, status, stream, tile_group, N);
+    return dispatch<EPI_GATED, float>(bn, mw, mx, (float*)C, ldc, T, N, K, half, 1, mode == 3, status, stream, tile_group, N);
   return LLM_ERR_UNSUPPORTED;
 }
 

@@ -115,12 +115,12 @@ template <int STAGES, int EPI, typename TC>
 __global__ void __launch_bounds__(192, 1) gemm_pair_kernel(
     const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
     const __grid_constant__ CUtensorMap map_c, int T, int N, int K, int half, int m_tiles, int n_tiles,
-    int ksplits, int* __restrict__ status) {
-  constexpr int FEAT = EPI == EPI_GATED ? 64 : TILE_M;     // output features of this CTA per tile
+    int ksplits, float act_limit, int* __restrict__ status) {
+  constexpr bool GATED = gated_epilogue(EPI);
+  constexpr int FEAT = GATED ? 64 : TILE_M;     // output features of this CTA per tile
   extern __shared__ uint8_t raw[];
   auto& sm = *reinterpret_cast<PairStorage<STAGES, FEAT, TC>*>(
       (reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
-  pdl_trigger();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const uint32_t rank = cluster_rank();
   const bool leader = rank == 0;
@@ -158,6 +158,7 @@ __global__ void __launch_bounds__(192, 1) gemm_pair_kernel(
   pair_sync();               // both CTAs' barriers exist before either signals the other
   tc_fence_after();
   const uint32_t tmem = sm.tmem_base;
+  pdl_trigger();             // after the allocation, as in the one-CTA kernel
 
   if (warp == 0 && lane == 0) {
     // ------------------------------------------------------------------ producer (both CTAs)
@@ -177,7 +178,7 @@ __global__ void __launch_bounds__(192, 1) gemm_pair_kernel(
       const int tile = work % tiles, ks = work / tiles;
       const int kb0 = (int)((long long)ks * nkb / ksplits), kb1 = (int)((long long)(ks + 1) * nkb / ksplits);
       const int f0 = (tile / n_tiles) * (2 * FEAT) + (int)rank * FEAT;      // first output feature
-      const int row0 = EPI == EPI_GATED ? 2 * f0 : f0;                      // first weight row
+      const int row0 = GATED ? 2 * f0 : f0;                      // first weight row
       const int t0 = (tile % n_tiles) * BN + (int)rank * HALF_N;
       int kb = kb0;
       if (first) {
@@ -258,11 +259,16 @@ __global__ void __launch_bounds__(192, 1) gemm_pair_kernel(
           uint32_t v[16];
           tmem_ld16(acc + (uint32_t)(c + h * 16), v);
           tmem_ld_wait();
-          if (EPI == EPI_GATED) {
+          if (GATED) {
             const int f = q * 16 + (lane & 15);
             const int col0 = h * 16 + (lane < 16 ? 0 : 8);
             float r[8];
-            gated_columns<TC>(v, lane, r);
+            if (EPI == EPI_CLAMPED) {
+              const float one[8] = {1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f};
+              clamped_columns<TC>(v, lane, act_limit, one, r);
+            } else {
+              gated_columns<TC>(v, lane, r);
+            }
 #pragma unroll
             for (int i = 0; i < 8; ++i) stage_out[(col0 + i) * FEAT + f] = from_f32<TC>(r[i]);
           } else {
@@ -308,8 +314,9 @@ __global__ void __launch_bounds__(192, 1) gemm_pair_kernel(
 
 template <int STAGES, int EPI, typename TC>
 int launch(const CUtensorMap& mw, const CUtensorMap& mx, const CUtensorMap& mc, int T, int N, int K, int half,
-           int sm_count, int* status, cudaStream_t stream) {
-  constexpr int FEAT = EPI == EPI_GATED ? 64 : TILE_M;
+           int sm_count, int* status, cudaStream_t stream, float act_limit = 0.f) {
+  constexpr bool GATED = gated_epilogue(EPI);
+  constexpr int FEAT = GATED ? 64 : TILE_M;
   auto kernel = gemm_pair_kernel<STAGES, EPI, TC>;
   constexpr int smem = (int)sizeof(PairStorage<STAGES, FEAT, TC>) + 1024;
   static_assert(smem <= 227 * 1024, "the stages and output chunks fit one SM");
@@ -319,7 +326,7 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mx, const CUtensorMap& mc, 
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  const int limit = EPI == EPI_GATED ? half : N;
+  const int limit = GATED ? half : N;
   const int m_tiles = (limit + 2 * FEAT - 1) / (2 * FEAT), n_tiles = (T + BN - 1) / BN;
   cudaLaunchConfig_t cfg = {};
   cfg.blockDim = dim3(192);
@@ -367,11 +374,11 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mx, const CUtensorMap& mc, 
   // directly behind the rotation kernel the pair kernel starts only when that kernel is done
   cfg.numAttrs = (g_llm_pdl && !g_llm_after_rotation) ? 2 : 1;
   g_llm_after_rotation = 0;
-  return (int)cudaLaunchKernelEx(&cfg, kernel, mw, mx, mc, T, N, K, half, m_tiles, n_tiles, ksplits, status);
+  return (int)cudaLaunchKernelEx(&cfg, kernel, mw, mx, mc, T, N, K, half, m_tiles, n_tiles, ksplits, act_limit, status);
 }
 }  // namespace
 
-// The pair kernel for bfloat16 X [T][K], W [N][K]; modes 0, 1 and 3 of llm_gemm_tcgen05 (no K
+// The pair kernel for bfloat16 X [T][K], W [N][K]; modes 0, 1, 3 and 4 of llm_gemm_tcgen05 (no K
 // split; the gated form only with interleaved rows).  Returns LLM_ERR_UNSUPPORTED when the output
 // cannot be written by TMA or the mode is not one of these: the caller then uses the one-CTA kernel.
 int g_llm_pair = 1;   // 0: the dispatcher keeps to the one-CTA kernels (for comparisons)
@@ -380,7 +387,7 @@ LLM_EXPORT void llm_set_pair_ksplits(int n) { g_llm_pair_ksplits = n; }
 LLM_EXPORT void llm_set_pair(int on) { g_llm_pair = on ? 1 : 0; }
 
 int llm_gemm_tcgen05_pair(const void* X, const void* W, void* C, int c_dtype, int T, int N, int K, int lda,
-                          int ldw, int ldc, int mode, int half, int* status, cudaStream_t stream) {
+                          int ldw, int ldc, int mode, int half, float limit, int* status, cudaStream_t stream) {
   if (!g_llm_pair) return LLM_ERR_UNSUPPORTED;
   static int sm_count = 0;
   if (!sm_count) {
@@ -389,14 +396,14 @@ int llm_gemm_tcgen05_pair(const void* X, const void* W, void* C, int c_dtype, in
     cudaDeviceGetAttribute(&sm_count, cudaDevAttrMultiProcessorCount, dev);
     if (sm_count <= 0) sm_count = 148;
   }
-  if (mode != 0 && mode != 1 && mode != 3) return LLM_ERR_UNSUPPORTED;
+  if (mode != 0 && mode != 1 && mode != 3 && mode != 4) return LLM_ERR_UNSUPPORTED;
   const int esize = c_dtype == LLM_F32 ? 4 : 2;
   if (((uintptr_t)C & 15) || ((size_t)ldc * esize) % 16) return LLM_ERR_UNSUPPORTED;
   CUtensorMap mw, mx, mc;
   if (!llm_tensor_map(W, N, K, ldw, TILE_M, TILE_K, 0, &mw)) return LLM_ERR_UNSUPPORTED;
   if (!llm_tensor_map(X, T, K, lda, HALF_N, TILE_K, 0, &mx)) return LLM_ERR_UNSUPPORTED;
-  const int out_cols = mode == 3 ? half : N;
-  if (!llm_tensor_map(C, T, out_cols, ldc, CH, mode == 3 ? 64 : TILE_M, c_dtype == LLM_F32 ? 2 : 1, &mc))
+  const int out_cols = mode >= 3 ? half : N;
+  if (!llm_tensor_map(C, T, out_cols, ldc, CH, mode >= 3 ? 64 : TILE_M, c_dtype == LLM_F32 ? 2 : 1, &mc))
     return LLM_ERR_UNSUPPORTED;
   if (mode == 0) {
     if (c_dtype == LLM_F32) return launch<5, EPI_STORE, float>(mw, mx, mc, T, N, K, half, sm_count, status, stream);
@@ -405,6 +412,9 @@ int llm_gemm_tcgen05_pair(const void* X, const void* W, void* C, int c_dtype, in
     if (c_dtype == LLM_F32) return launch<5, EPI_ACCUM, float>(mw, mx, mc, T, N, K, half, sm_count, status, stream);
   } else {
     if (N != 2 * half || half % 16) return LLM_ERR_ARGUMENT;
+    if (mode == 4)
+      return c_dtype == LLM_BF16 ? launch<6, EPI_CLAMPED, bf16>(mw, mx, mc, T, N, K, half, sm_count, status, stream, limit)
+                                 : LLM_ERR_UNSUPPORTED;
     if (c_dtype == LLM_BF16) return launch<6, EPI_GATED, bf16>(mw, mx, mc, T, N, K, half, sm_count, status, stream);
     if (c_dtype == LLM_F32) return launch<6, EPI_GATED, float>(mw, mx, mc, T, N, K, half, sm_count, status, stream);
   }

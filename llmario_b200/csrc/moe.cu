@@ -25,7 +25,8 @@ constexpr int MAX_TOP = 16;
 // the weights are a softmax in which only the chosen logits take part.  mode 1: scores are the
 // softmax over all E outputs; the choice goes by score + corr[e] (the same tie rule), the weight
 // of a chosen expert is its score, not renormalised.  mode 2: as mode 1, but the weights are the
-// chosen scores over their sum (+ 1e-20), times `wscale`.
+// chosen scores over their sum (+ 1e-20), times `wscale`.  mode 3: the choice as in mode 0 (the sigmoid
+// keeps the order of the logits); the weight of a chosen expert is the sigmoid of its own logit.
 __device__ __forceinline__ void choose_row(const float* zr, int E, int top, int mode, const float* __restrict__ corr,
                                            int lane, int* __restrict__ ids, float* __restrict__ wts,
                                            float wscale = 1.f) {
@@ -71,6 +72,10 @@ __device__ __forceinline__ void choose_row(const float* zr, int E, int top, int 
         const float f = wscale / (chosen + 1e-20f);
         for (int k = 0; k < top; ++k) wts[k] *= f;
       }
+      return;
+    }
+    if (mode == 3) {
+      for (int k = 0; k < top; ++k) ids[k] = pick[k], wts[k] = 1.f / (1.f + expf(-best[k]));
       return;
     }
     float sum = 0.f;       // best[0] is the largest
@@ -188,12 +193,15 @@ template <> __device__ __forceinline__ float dot_row<bf16>(const bf16* __restric
 
 // grid (rows * top, ff tiles of 8); a block stages its row of h in shared memory, a warp makes
 // two features.  gate_up: [E][2 ff][width], gate rows first; kind 3 (an expert without a gate,
-// act = max(W_up h, 0)^2): [E][ff][width].
+// act = max(W_up h, 0)^2): [E][ff][width].  in_wts: a factor per item on the expert's input (applied to
+// the products, in 32-bit), or null.  interleaved: an expert's rows stand as 16 gate rows, their 16 up
+// rows, the next 16 gate rows, ... (the order of the grouped tensor-core product).
 template <typename T>
 __global__ void __launch_bounds__(128) moe_gate_up_rows_kernel(const T* __restrict__ h, const T* __restrict__ gate_up,
                                                                const int* __restrict__ ids, T* __restrict__ act,
                                                                int width, int ff, int top, int E, int kind,
-                                                               float limit) {
+                                                               float limit, const float* __restrict__ in_wts,
+                                                               int interleaved) {
   extern __shared__ float h_s[];
   pdl_trigger();
   pdl_wait();
@@ -203,15 +211,18 @@ __global__ void __launch_bounds__(128) moe_gate_up_rows_kernel(const T* __restri
   for (int i = threadIdx.x; i < width; i += blockDim.x) h_s[i] = to_f32(h[(size_t)r * width + i]);
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const float ws = in_wts ? in_wts[item] : 1.f;
   const T* we = gate_up + (size_t)e * (kind == 3 ? 1 : 2) * ff * width;
   for (int f = blockIdx.y * 8 + warp; f < min(ff, blockIdx.y * 8 + 8); f += 4) {
-    const float g = dot_row<T>(we + (size_t)f * width, h_s, width, lane);
+    const int g_row = interleaved ? (f >> 4) * 32 + (f & 15) : f;
+    const float g = ws * dot_row<T>(we + (size_t)g_row * width, h_s, width, lane);
     if (kind == 3) {
       const float p = fmaxf(g, 0.f);
       if (lane == 0) act[(size_t)item * ff + f] = from_f32<T>(p * p);
       continue;
     }
-    const float u = dot_row<T>(we + (size_t)(ff + f) * width, h_s, width, lane);
+    const int u_row = interleaved ? g_row + 16 : ff + f;
+    const float u = ws * dot_row<T>(we + (size_t)u_row * width, h_s, width, lane);
     if (lane == 0) {
       float y;
       if (kind == 2) {       // the gate bounded above, the other half on both sides and one added to it
@@ -251,7 +262,7 @@ __global__ void __launch_bounds__(128) moe_down_rows_kernel(const T* __restrict_
       // an expert behind the E with matrices is the identity: its output is the input itself
       const float d = e >= 0 && e < E ? dot_row<T>(down + ((size_t)e * width + c) * ff, a_s + (size_t)k * ff, ff, lane)
                                       : to_f32(h[(size_t)r * width + c]);
-      sum = fmaf(wts[(size_t)r * top + k], d, sum);
+      sum = fmaf(wts ? wts[(size_t)r * top + k] : 1.f, d, sum);
     }
     if (lane == 0) {
       if (shared) {
@@ -297,15 +308,18 @@ __global__ void __launch_bounds__(1024) moe_align_kernel(const int* __restrict__
   }
 }
 
-// xp[pos[i]][:] = h[i / top][:]
+// xp[pos[i]][:] = h[i / top][:]; with row_scale: row_scale[pos[i]] = wts[i] beside it
 template <typename T>
 __global__ void __launch_bounds__(128) moe_gather_kernel(const T* __restrict__ h, const int* __restrict__ pos,
                                                          T* __restrict__ xp, int width, int top,
-                                                         const int* __restrict__ ids, int E) {
+                                                         const int* __restrict__ ids, int E,
+                                                         const float* __restrict__ wts,
+                                                         float* __restrict__ row_scale) {
   pdl_trigger();
   pdl_wait();
   const int i = blockIdx.x;
   if (ids && (ids[i] < 0 || ids[i] >= E)) return;      // an identity expert has no row in the buffer
+  if (row_scale && threadIdx.x == 0) row_scale[pos[i]] = wts[i];
   const T* src = h + (size_t)(i / top) * width;
   T* dst = xp + (size_t)pos[i] * width;
   if ((width * sizeof(T)) % 16 == 0 && (((uintptr_t)h | (uintptr_t)xp) & 15) == 0) {
@@ -318,6 +332,7 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const T* __restrict__ h
 }
 
 // y[r][c] (+)= sum_k wts[r][k] * d[pos[r * top + k]][c]  (+ sigmoid(gate[r]) * shared[r][c]), k ascending
+// (wts null: all ones)
 __global__ void __launch_bounds__(256) moe_combine_kernel(const float* __restrict__ d, const int* __restrict__ pos,
                                                           const float* __restrict__ wts,
                                                           float* __restrict__ shared,
@@ -337,7 +352,7 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const float* __restric
       const float v = !identity ? d[(size_t)pos[(size_t)r * top + k] * width + c]
                       : x_dtype == LLM_BF16 ? to_f32(((const bf16*)x_id)[(size_t)r * x_stride + c])
                                             : ((const float*)x_id)[(size_t)r * x_stride + c];
-      sum = fmaf(wts[(size_t)r * top + k], v, sum);
+      sum = fmaf(wts ? wts[(size_t)r * top + k] : 1.f, v, sum);
     }
     if (shared) {
       sum = fmaf(g, shared[(size_t)r * width + c], sum);
@@ -357,16 +372,19 @@ LLM_EXPORT int llm_moe_align(const int* ids, int n_pairs, int E, int bn, int n_t
                     pos, tile_group);
 }
 
-// (ids with E: pairs whose expert is not one of the E with matrices are left out)
+// (ids with E: pairs whose expert is not one of the E with matrices are left out; wts with row_scale:
+// the pairs' weights are put in the order of the buffer's rows)
 LLM_EXPORT int llm_moe_gather(const void* h, const int* pos, void* xp, int dtype, int n_pairs, int width, int top,
-                              const int* ids, int E, cudaStream_t stream) {
+                              const int* ids, int E, const float* wts, float* row_scale,
+                              cudaStream_t stream) {
   if (n_pairs <= 0) return 0;
+  if ((wts != nullptr) != (row_scale != nullptr)) return LLM_ERR_ARGUMENT;
   if (dtype == LLM_F32)
     return launch_pdl(moe_gather_kernel<float>, n_pairs, 128, 0, stream, (const float*)h, pos, (float*)xp, width, top,
-                      ids, E);
+                      ids, E, wts, row_scale);
   if (dtype == LLM_BF16)
     return launch_pdl(moe_gather_kernel<bf16>, n_pairs, 128, 0, stream, (const bf16*)h, pos, (bf16*)xp, width, top,
-                      ids, E);
+                      ids, E, wts, row_scale);
   return LLM_ERR_UNSUPPORTED;
 }
 
@@ -389,7 +407,7 @@ LLM_EXPORT int llm_moe_router_scaled(const void* h, int dtype, const float* w, c
                                      int z_stride, int rows, int width, int E, int n_out, int top, int mode,
                                      const float* corr, int* ids, float* wts, float wscale, cudaStream_t stream) {
   if (rows <= 0) return 0;
-  if (top < 1 || top > MAX_TOP || top > E || n_out < E || mode < 0 || mode > 2) return LLM_ERR_UNSUPPORTED;
+  if (top < 1 || top > MAX_TOP || top > E || n_out < E || mode < 0 || mode > 3) return LLM_ERR_UNSUPPORTED;
   if ((size_t)(width + n_out) * 4 > 200 * 1024) return LLM_ERR_UNSUPPORTED;
   // many rows: four to a block, so that a block reads the router's rows once for four tokens
   const bool four = rows >= 256 && (size_t)4 * (width + n_out) * 4 <= 200 * 1024;
@@ -425,7 +443,7 @@ LLM_EXPORT int llm_moe_router(const void* h, int dtype, const float* w, const fl
 LLM_EXPORT int llm_moe_route_scaled(const float* z, int z_stride, int rows, int E, int top, int mode,
                                     const float* corr, int* ids, float* wts, float wscale, cudaStream_t stream) {
   if (rows <= 0) return 0;
-  if (top < 1 || top > MAX_TOP || top > E || mode < 0 || mode > 2) return LLM_ERR_UNSUPPORTED;
+  if (top < 1 || top > MAX_TOP || top > E || mode < 0 || mode > 3) return LLM_ERR_UNSUPPORTED;
   return launch_pdl(moe_route_kernel, (rows + 3) / 4, 128, 0, stream, z, z_stride, rows, E, top, mode, corr, ids,
                     wts, wscale);
 }
@@ -436,11 +454,14 @@ LLM_EXPORT int llm_moe_route(const float* z, int z_stride, int rows, int E, int 
 }
 
 // E: experts with matrices (a pair whose expert is not one of them is left out); kind 0: silu(g) u,
-// 2: the clamped form with `limit` (see activations.cu), 3: no gate, max(u, 0)^2 with gate_up [E][ff][width]
+// 2: the clamped form with `limit` (see activations.cu), 3: no gate, max(u, 0)^2 with gate_up [E][ff][width];
+// in_wts [rows][top]: a factor on the input of each (row, chosen expert), or null; interleaved: the order of
+// an expert's gate and up rows (16 and 16), ff a multiple of 16
 LLM_EXPORT int llm_moe_gate_up_rows(const void* h, const void* gate_up, const int* ids, void* act, int dtype,
                                     int rows, int width, int ff, int top, int E, int kind, float limit,
-                                    cudaStream_t stream) {
+                                    const float* in_wts, int interleaved, cudaStream_t stream) {
   if (rows <= 0) return 0;
+  if (interleaved && (kind == 3 || ff % 16)) return LLM_ERR_ARGUMENT;
   if ((ff + 7) / 8 > 65535 || (size_t)width * 4 > 200 * 1024) return LLM_ERR_UNSUPPORTED;
   const dim3 grid(rows * top, (ff + 7) / 8);
   const size_t smem = (size_t)width * 4;
@@ -448,13 +469,14 @@ LLM_EXPORT int llm_moe_gate_up_rows(const void* h, const void* gate_up, const in
     if (smem > 48 * 1024)
       cudaFuncSetAttribute(moe_gate_up_rows_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     return launch_pdl(moe_gate_up_rows_kernel<float>, grid, 128, smem, stream, (const float*)h,
-                      (const float*)gate_up, ids, (float*)act, width, ff, top, E, kind, limit);
+                      (const float*)gate_up, ids, (float*)act, width, ff, top, E, kind, limit, in_wts,
+                      interleaved);
   }
   if (dtype == LLM_BF16) {
     if (smem > 48 * 1024)
       cudaFuncSetAttribute(moe_gate_up_rows_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     return launch_pdl(moe_gate_up_rows_kernel<bf16>, grid, 128, smem, stream, (const bf16*)h, (const bf16*)gate_up,
-                      ids, (bf16*)act, width, ff, top, E, kind, limit);
+                      ids, (bf16*)act, width, ff, top, E, kind, limit, in_wts, interleaved);
   }
   return LLM_ERR_UNSUPPORTED;
 }

@@ -9,7 +9,9 @@ constexpr int TILE_K = 64;        // bf16 elements per stage row: 128 bytes, one
 constexpr int UMMA_K = 16;
 
 
-enum Epilogue : int { EPI_STORE = 0, EPI_ACCUM = 1, EPI_GATED = 2 };
+// (the gated ones: silu(g) u, and the clamped form of clamped_swish_mul below)
+enum Epilogue : int { EPI_STORE = 0, EPI_ACCUM = 1, EPI_GATED = 2, EPI_CLAMPED = 3 };
+constexpr bool gated_epilogue(int epi) { return epi == EPI_GATED || epi == EPI_CLAMPED; }
 
 __device__ __forceinline__ void tma_load_2d(void* dst, const CUtensorMap* map, int x, int y, uint64_t* bar) {
   asm volatile(
@@ -62,6 +64,13 @@ template <typename TC> __device__ __forceinline__ float silu_mul(float g, float 
   if (sizeof(TC) == 2) return __fdividef(g, 1.0f + __expf(-g)) * u;
   return g / (1.0f + __expf(-g)) * u;
 }
+// g sigmoid(1.702 g) (u + 1) with g bounded above by `limit` and u on both sides, in 32-bit
+template <typename TC> __device__ __forceinline__ float clamped_swish_mul(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit) + 1.0f;
+  if (sizeof(TC) == 2) return __fdividef(g, 1.0f + __expf(-1.702f * g)) * u;
+  return g / (1.0f + __expf(-1.702f * g)) * u;
+}
 // Gated epilogue of 16 accumulator columns v[0..15].  In each warp lanes 0..15 hold gate rows and
 // lanes 16..31 the up rows of the same 16 features.  Both halves of the warp work: lane L < 16
 // and lane L + 16 swap half of their columns, so that L computes columns 0..7 of its feature and
@@ -74,6 +83,20 @@ template <typename TC> __device__ __forceinline__ void gated_columns(const uint3
     const float send = __uint_as_float(low ? v[8 + i] : v[i]);
     const float got = __shfl_xor_sync(0xffffffffu, send, 16);
     out[i] = low ? silu_mul<TC>(keep, got) : silu_mul<TC>(got, keep);
+  }
+}
+// The same for the clamped form; scale[i] multiplies gate and up of output column i first.
+template <typename TC>
+__device__ __forceinline__ void clamped_columns(const uint32_t* v, int lane, float limit, const float* scale,
+                                                float* out) {
+  const bool low = lane < 16;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const float keep = __uint_as_float(low ? v[i] : v[8 + i]);
+    const float send = __uint_as_float(low ? v[8 + i] : v[i]);
+    const float got = __shfl_xor_sync(0xffffffffu, send, 16);
+    const float g = (low ? keep : got) * scale[i], u = (low ? got : keep) * scale[i];
+    out[i] = clamped_swish_mul<TC>(g, u, limit);
   }
 }
 

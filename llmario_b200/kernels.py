@@ -107,11 +107,12 @@ def _signatures():
         "llm_moe_route": [P, I, I, I, I, I, P, P, P, P],
         "llm_moe_router": [P, I, P, P, P, I, I, I, I, I, I, I, P, P, P, P],
         "llm_moe_align": [P, I, I, I, I, P, P, P],
-        "llm_moe_gather": [P, P, P, I, I, I, I, P, I, P],
+        "llm_moe_gather": [P, P, P, I, I, I, I, P, I, P, P, P],
         "llm_moe_combine": [P, P, P, P, P, I, P, I, I, I, I, I, P, I, P, I, I, P],
-        "llm_gemm_tcgen05_grouped": [P, P, P, I, I, I, I, I, I, I, I, I, I, I, P, P, P],
+        "llm_gemm_tcgen05_grouped": [P, P, P, I, I, I, I, I, I, I, I, I, I, I, P, F, P, P, P],
+        "llm_gemm_tcgen05_clamped": [P, P, P, I, I, I, I, I, I, I, F, P, P],
         "llm_gemm_tcgen05_batched": [P, P, P, I, I, I, I, I, I, I, I, I, I, I, P, P],
-        "llm_moe_gate_up_rows": [P, P, P, P, I, I, I, I, I, I, I, F, P],
+        "llm_moe_gate_up_rows": [P, P, P, P, I, I, I, I, I, I, I, F, P, I, P],
         "llm_moe_down_rows": [P, P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, P, P],
         "llm_causal_conv_silu": [P, I, P, P, P, L, P, P, I, I, I, P, I, I, I, P],
         "llm_gated_group_norm": [P, I, P, I, P, I, P, I, P, I, P, I, I, I, I, I, F, I, P],
@@ -797,6 +798,9 @@ def selftest_wait_gives_up(device, limit_cycles: int = 20000) -> None:
            "selftest_wait_gives_up")
 
 
+PAIR_MIN_ROWS = 512       # steps of so many rows take their products on CTA pairs (token_tile)
+
+
 def token_tile(rows: int) -> int:
     """Tokens per tile of the tensor-core product: the smallest tile that holds the rows, 256
     (the persistent kernel) once there are enough rows to fill the GPU with such tiles."""
@@ -949,6 +953,22 @@ def gate_up_silu(ctx, h: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tenso
     gu = ctx.buffer("ffn.gate_up", (rows, 2 * ff), torch.float32)
     linear(h, w_gate_up, gu)
     silu_mul(gu, act)
+
+
+def gate_up_clamped(h: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor,
+                    limit: float) -> None:
+    """act = g sigmoid(1.702 g) (u + 1) with g = min(h Wg^T, limit), u = clamp(h Wu^T, +-limit) in
+    one tensor-core product; ``w_gate_up`` [2 ff, hidden] as alternating blocks of 16 gate and 16
+    up rows, everything bfloat16."""
+    if not _tc_ok(h, w_gate_up, act) or act.dtype != torch.bfloat16:
+        raise KernelError("interleaved gate/up weights need the tensor-core product")
+    rows, ff = act.shape
+    K = h.shape[1]
+    _check(lib().llm_gemm_tcgen05_clamped(_ptr(h), _ptr(w_gate_up), _ptr(act), rows, ff, K,
+                                          h.stride(0), w_gate_up.stride(0), act.stride(0),
+                                          token_tile(rows), float(limit),
+                                          _ptr(tc_status(h.device)), _stream()),
+           "gate_up_clamped")
 
 
 FLASH_HEAD_DIMS = (32, 64, 128)
@@ -1443,16 +1463,16 @@ def head_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
                                        out.stride(1), _stream()), "head_linear")
 
 
-ROUTE_SOFTMAX_CHOSEN, ROUTE_SOFTMAX_ALL, ROUTE_SOFTMAX_ALL_RENORMED = 0, 1, 2
+ROUTE_SOFTMAX_CHOSEN, ROUTE_SOFTMAX_ALL, ROUTE_SOFTMAX_ALL_RENORMED, ROUTE_SIGMOID = 0, 1, 2, 3
 ROUTE_MODES = {"softmax_chosen": ROUTE_SOFTMAX_CHOSEN, "softmax_all": ROUTE_SOFTMAX_ALL,
-               "softmax_all_renormed": ROUTE_SOFTMAX_ALL_RENORMED}
+               "softmax_all_renormed": ROUTE_SOFTMAX_ALL_RENORMED, "sigmoid": ROUTE_SIGMOID}
 
 
 def _route_mode(scores: str, correction: Optional[torch.Tensor], experts: int) -> int:
     if scores not in ROUTE_MODES:
         raise KernelError(f"router scores '{scores}' ({', '.join(ROUTE_MODES)})")
     if correction is not None:
-        assert scores != "softmax_chosen" and correction.dtype == torch.float32
+        assert scores not in ("softmax_chosen", "sigmoid") and correction.dtype == torch.float32
         assert correction.is_contiguous() and correction.numel() == experts
     return ROUTE_MODES[scores]
 
@@ -1465,7 +1485,8 @@ def moe_route(z: torch.Tensor, experts: int, top: int, ids: torch.Tensor, wts: t
     ``scores="softmax_all"``: the scores are the softmax over all ``experts`` logits, the choice
     goes by score + ``correction`` (float32 [experts], optional), and a chosen expert's weight is
     its score, not renormalised.  ``"softmax_all_renormed"``: the same choice; the weights are the
-    chosen scores over their sum (+ 1e-20), times ``weight_scale``."""
+    chosen scores over their sum (+ 1e-20), times ``weight_scale``.  ``"sigmoid"``: the largest
+    logits; the weight of a chosen expert is the sigmoid of its logit."""
     _cuda(z, ids, wts, correction)
     mode = _route_mode(scores, correction, experts)
     rows = z.shape[0]
@@ -1502,13 +1523,20 @@ def moe_router(h: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], e
 
 
 def moe_gate_up_rows(h: torch.Tensor, gate_up: torch.Tensor, ids: torch.Tensor,
-                     act: torch.Tensor, activation: str = "silu", limit: float = 0.0) -> None:
+                     act: torch.Tensor, activation: str = "silu", limit: float = 0.0,
+                     input_weights: Optional[torch.Tensor] = None,
+                     interleaved: bool = False) -> None:
     """act[r, k] = silu(Wg_e h_r) * (Wu_e h_r), e = ids[r, k]; gate_up [E, 2 ff, width].  With
     ``activation="clamped_swish"`` the gated form of that name (see :func:`gated_act`).  A pair
     whose expert is not one of the E with matrices is left out.  ``activation="relu_squared"``:
     experts without a gate, ``gate_up`` [E, ff, width] holds their up matrices and
-    act[r, k] = max(Wu_e h_r, 0)^2."""
-    _cuda(h, gate_up, ids, act)
+    act[r, k] = max(Wu_e h_r, 0)^2.  ``input_weights`` (float32 [rows, top]): expert ids[r, k]
+    reads input_weights[r, k] h_r.  ``interleaved``: an expert's rows stand as 16 gate rows, their
+    16 up rows, the next 16 gate rows, ..."""
+    _cuda(h, gate_up, ids, act, input_weights)
+    assert input_weights is None or (input_weights.dtype == torch.float32
+                                     and input_weights.is_contiguous()
+                                     and input_weights.shape == ids.shape)
     if activation not in ("silu", "clamped_swish", "relu_squared"):
         raise KernelError(f"routed experts have no activation '{activation}'")
     rows, width = h.shape
@@ -1519,17 +1547,19 @@ def moe_gate_up_rows(h: torch.Tensor, gate_up: torch.Tensor, ids: torch.Tensor,
     _check(lib().llm_moe_gate_up_rows(_ptr(h), _ptr(gate_up), _ptr(ids), _ptr(act), _dt(h), rows,
                                       width, ff, top, gate_up.shape[0],
                                       {**ACTIVATIONS, **PLAIN_ACTIVATIONS}[activation],
-                                      float(limit), _stream()), "moe_gate_up_rows")
+                                      float(limit), _ptr(input_weights), int(interleaved),
+                                      _stream()), "moe_gate_up_rows")
 
 
-def moe_down_rows(act: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor,
+def moe_down_rows(act: torch.Tensor, down: torch.Tensor, ids: torch.Tensor,
+                  wts: Optional[torch.Tensor],
                   y: torch.Tensor, accumulate: bool, shared: Optional[torch.Tensor] = None,
                   shared_gate: Optional[torch.Tensor] = None, clear_shared: bool = False,
                   identity_input: Optional[torch.Tensor] = None) -> None:
     """y[r] (+)= sum_k wts[r, k] Wd_e act[r, k] (+ sigmoid(shared_gate[r]) shared[r]);
     down [E, width, ff]; y, shared float32 [rows, width]; shared_gate float32 [rows] (strided).
     ``identity_input`` ([rows, width], act's type): an expert index of E or more is an identity
-    expert, whose output is that row."""
+    expert, whose output is that row.  ``wts`` None: every weight is one."""
     _cuda(act, down, ids, wts, y, shared, shared_gate, identity_input)
     if identity_input is not None:
         assert identity_input.dtype == act.dtype and identity_input.is_contiguous()
@@ -1577,29 +1607,37 @@ def moe_align(ids: torch.Tensor, experts: int, bn: int, pos: torch.Tensor,
 
 
 def moe_gather(h: torch.Tensor, pos: torch.Tensor, xp: torch.Tensor, top: int,
-               ids: Optional[torch.Tensor] = None, experts: int = 0) -> None:
-    """xp[pos[i]] = h[i // top] (with ``ids``: only for pairs whose expert is below ``experts``)."""
-    _cuda(h, pos, xp, ids)
+               ids: Optional[torch.Tensor] = None, experts: int = 0,
+               wts: Optional[torch.Tensor] = None,
+               row_scale: Optional[torch.Tensor] = None) -> None:
+    """xp[pos[i]] = h[i // top] (with ``ids``: only for pairs whose expert is below ``experts``).
+    ``wts`` with ``row_scale`` (float32): row_scale[pos[i]] = wts[i] beside it."""
+    _cuda(h, pos, xp, ids, wts, row_scale)
+    if wts is not None:
+        assert wts.dtype == row_scale.dtype == torch.float32 and wts.is_contiguous()
+        assert wts.numel() == pos.numel() and row_scale.numel() >= xp.shape[0]
     assert h.is_contiguous() and xp.is_contiguous() and h.dtype == xp.dtype
     assert h.shape[1] == xp.shape[1] and pos.numel() == h.shape[0] * top
     _check(lib().llm_moe_gather(_ptr(h), _ptr(pos), _ptr(xp), _dt(h), pos.numel(), h.shape[1], top,
-                                _ptr(ids), int(experts), _stream()), "moe_gather")
+                                _ptr(ids), int(experts), _ptr(wts), _ptr(row_scale), _stream()),
+           "moe_gather")
 
 
-def moe_combine(d: torch.Tensor, pos: torch.Tensor, wts: torch.Tensor, y: torch.Tensor,
-                accumulate: bool, shared: Optional[torch.Tensor] = None,
+def moe_combine(d: torch.Tensor, pos: torch.Tensor, wts: Optional[torch.Tensor],
+                y: torch.Tensor, accumulate: bool, shared: Optional[torch.Tensor] = None,
                 shared_gate: Optional[torch.Tensor] = None, clear_shared: bool = False,
                 ids: Optional[torch.Tensor] = None, experts: int = 0,
                 identity_input: Optional[torch.Tensor] = None) -> None:
     """y[r] (+)= sum_k wts[r, k] d[pos[r, k]] (+ sigmoid(shared_gate[r]) shared[r]).  With
     ``ids``: a pair whose expert is ``experts`` or more is an identity expert, whose output is
-    the row of ``identity_input`` ([rows, width])."""
+    the row of ``identity_input`` ([rows, width]).  ``wts`` None: every weight is one."""
     _cuda(d, pos, wts, y, shared, shared_gate, ids, identity_input)
     if ids is not None:
         assert identity_input is not None and identity_input.stride(1) == 1
-    rows, top = wts.shape
-    width = y.shape[1]
-    assert d.dtype == y.dtype == wts.dtype == torch.float32 and d.is_contiguous()
+    rows, width = y.shape
+    top = pos.numel() // rows
+    assert d.dtype == y.dtype == torch.float32 and d.is_contiguous()
+    assert wts is None or (wts.dtype == torch.float32 and wts.shape == (rows, top))
     assert y.is_contiguous() and d.shape[1] == width and pos.numel() == rows * top
     if shared is not None:
         assert shared.dtype == torch.float32 and shared.is_contiguous()
@@ -1614,16 +1652,28 @@ def moe_combine(d: torch.Tensor, pos: torch.Tensor, wts: torch.Tensor, y: torch.
 
 
 def gemm_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_group: torch.Tensor,
-                 bn: int, gated: bool) -> None:
+                 bn: int, gated: bool, interleaved: bool = False, activation: str = "silu",
+                 limit: float = 0.0, row_scale: Optional[torch.Tensor] = None) -> None:
     """The tensor-core product with a matrix per tile of ``bn`` rows of ``a``: tile t uses
     ``w[tile_group[t]]`` (w [groups, N, K] bfloat16; a negative entry leaves the tile out).
-    ``gated``: w[g] = [gate; up] and out = silu(a gate^T) * (a up^T) ([rows, N / 2])."""
-    _cuda(a, w, out, tile_group)
+    ``gated``: w[g] = [gate; up] and out = silu(a gate^T) * (a up^T) ([rows, N / 2]);
+    ``interleaved``: w[g] has its rows as 16 gate rows, their 16 up rows, ...; with interleaved
+    rows ``activation="clamped_swish"`` (``limit``; see :func:`gated_act`) and ``row_scale``
+    (float32 [rows], a factor per row on both products in front of it) are there as well."""
+    _cuda(a, w, out, tile_group, row_scale)
+    mode = 0 if not gated else 2
+    if gated and interleaved:
+        mode = {"silu": 3, "clamped_swish": 4}[activation]
+    elif activation != "silu":
+        raise KernelError(f"the grouped product with rows [gate; up] has no '{activation}'")
+    assert row_scale is None or (mode == 4 and row_scale.dtype == torch.float32
+                                 and row_scale.numel() >= a.shape[0])
     T, K = a.shape
     G, N, _ = w.shape
     assert a.dtype == w.dtype == torch.bfloat16 and a.is_contiguous() and w.is_contiguous()
     assert out.stride(1) == 1 and tile_group.numel() * bn >= T
     _check(lib().llm_gemm_tcgen05_grouped(_ptr(a), _ptr(w), _ptr(out), _dt(out), T, N, K,
-                                          a.stride(0), K, out.stride(0), 2 if gated else 0,
+                                          a.stride(0), K, out.stride(0), mode,
                                           N // 2 if gated else 0, bn, G, _ptr(tile_group),
+                                          float(limit), _ptr(row_scale),
                                           _ptr(tc_status(a.device)), _stream()), "gemm_grouped")

@@ -4,6 +4,7 @@ sublayer's output, the one over several residual streams, and the one whose two 
 the same normed input (``x += mixer(norm(x)) + feed_forward(norm(x))``).  The residual stream ``x`` is 32-bit in every mode; the parts add into it."""
 from __future__ import annotations
 
+import contextlib
 from typing import Dict
 
 import torch
@@ -152,11 +153,20 @@ class HyperConnectionBlock:
     a layer's last sublayer is left to the block that runs next (or to the end of the step),
     which finds it under ``ctx.shared["streams.pending"]``.  Tensor roles: ``mixer_in`` [S],
     ``mixer_out`` [S], ``mixer_mix`` [S, S] (indexed [from, to]) and the same for
-    ``feed_forward_*``; a feed-forward of kind ``none`` leaves a layer with one sublayer."""
+    ``feed_forward_*``; a feed-forward of kind ``none`` leaves a layer with one sublayer.
+
+    With ``residual_scale`` (one stream, no tensors) the coefficients are the constants of
+    ``x += residual_scale * sublayer(norm(x))``."""
 
     def __init__(self, spec: PartSpec, layer: LayerSpec, weights: Dict[str, torch.Tensor],
                  dtype, device):
         self.streams = int(spec["streams"])
+        fixed = None
+        if spec.get("residual_scale") is not None:
+            if self.streams != 1:
+                raise ConfigError("hyper-connection block: residual_scale is for one stream")
+            fixed = tuple(torch.full((1,), v, dtype=torch.float32, device=device)
+                          for v in (1.0, float(spec["residual_scale"]), 1.0))   # in, out, mix
 
         def coef(role, shape):
             t = optional_tensor_of(spec, role, weights)
@@ -170,13 +180,13 @@ class HyperConnectionBlock:
         self.feed_forward = build_part("feed_forward", layer.feed_forward, weights, dtype,
                                        device)
         self.has_feed_forward = layer.feed_forward.kind != "none"
-        self.mixer_coef = (coef("mixer_in", (S,)), coef("mixer_out", (S,)),
-                           coef("mixer_mix", (S, S)))
+        self.mixer_coef = fixed or (coef("mixer_in", (S,)), coef("mixer_out", (S,)),
+                                    coef("mixer_mix", (S, S)))
         self.ffn_norm = self.ffn_coef = None
         if self.has_feed_forward:
             self.ffn_norm = build_part("norm", spec["feed_forward_norm"], weights, dtype, device)
-            self.ffn_coef = (coef("feed_forward_in", (S,)), coef("feed_forward_out", (S,)),
-                             coef("feed_forward_mix", (S, S)))
+            self.ffn_coef = fixed or (coef("feed_forward_in", (S,)), coef("feed_forward_out", (S,)),
+                                      coef("feed_forward_mix", (S, S)))
         for norm in (self.mixer_norm, self.ffn_norm):
             if norm is not None and type(norm) is not RmsNorm:
                 raise ConfigError("the hyper-connection block fuses an RMS norm with the mixing "
@@ -193,6 +203,16 @@ class HyperConnectionBlock:
         return graph_safe(self.mixer) and graph_safe(self.feed_forward)
 
     def forward(self, ctx: StepContext, call: BoundCall, xs: torch.Tensor) -> None:
+        # Steps of many rows take their products on CTA pairs.  As programmatic dependents of
+        # chains of small kernels such products have stopped making progress (once in a while, in
+        # models with mixers of several small kernels), and a step of many rows gains nothing from
+        # the overlap: its kernels start in plain stream order.
+        order = kernels.plain_stream_order() if ctx.rows >= kernels.PAIR_MIN_ROWS \
+            else contextlib.nullcontext()
+        with order:
+            self._forward(ctx, call, xs)
+
+    def _forward(self, ctx: StepContext, call: BoundCall, xs: torch.Tensor) -> None:
         if xs.dim() != 3 or xs.shape[0] != self.streams:
             raise RuntimeError(f"a hyper-connection block of {self.streams} streams was given a "
                                f"residual of shape {tuple(xs.shape)}")

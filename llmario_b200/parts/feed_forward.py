@@ -5,15 +5,19 @@ crates/engine/cpu/src/ops.rs:83-99).  Gate and up are one product over stacked r
 Beside it: the same form with a choice of activation and optional biases (kind ``gated``), and
 routed experts (kind ``moe``): a router's logits (32-bit) choose ``top`` of ``experts`` small
 silu-gated feed-forwards per token, whose outputs are summed with the softmax over the chosen
-logits as weights; an optional shared feed-forward is applied to all tokens and added with a
-per-token scalar weight, the sigmoid of one more projection of the input.  Options of the routed
+logits as weights; an optional shared feed-forward is applied to all tokens and added, as it is or
+(tensor role ``shared_gate``) with a per-token scalar weight, the sigmoid of one more projection of
+the input.  Options of the routed
 experts: ``scores: "softmax_all"`` (the scores are the softmax over all router outputs, the choice
 goes by score plus the tensor ``correction``, and a chosen expert's weight is its score, not
 renormalised); ``identity`` (the last so many router outputs are experts without matrices whose
 output is the input itself); ``activation: "clamped_swish"`` with ``limit``;
 ``scores: "softmax_all_renormed"`` (as ``softmax_all``, but the weights are the chosen scores over
 their sum, times ``weight_scale``); ``activation: "relu_squared"`` (experts without a gate,
-``W_down max(W_up h, 0)^2``: there are no ``gate<e>`` tensors).
+``W_down max(W_up h, 0)^2``: there are no ``gate<e>`` tensors); ``scores: "sigmoid"`` (the largest
+logits are chosen; a chosen expert's weight is the sigmoid of its logit, not renormalised);
+``weight_on: "input"`` (a chosen expert reads its weight times the token's input, and its output is
+added as it is).
 
 And a feed-forward without a gate (kind ``dense``): ``y = W_down act(W_up h)``."""
 from __future__ import annotations
@@ -28,6 +32,15 @@ from .base import StepContext, build_part, optional_tensor_of, register_part, te
 from .linear import Linear
 
 
+def interleaved_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+    """Gate and up rows as alternating blocks of 16: 16 gate rows, their 16 up rows, the next 16
+    gate rows, ... ([.., ff, k] each, ff a multiple of 16)."""
+    *lead, ff, k = gate.shape
+    both = torch.stack([gate.reshape(*lead, ff // 16, 16, k), up.reshape(*lead, ff // 16, 16, k)],
+                       dim=-3)
+    return both.reshape(*lead, 2 * ff, k).contiguous()
+
+
 class SwiGLU:
     graph_safe = True
 
@@ -40,9 +53,7 @@ class SwiGLU:
         # with gate and up of a feature in the same quarter of the accumulator.
         self.interleaved = kernels.gated_interleave_ok(gate, up)
         if self.interleaved:
-            ff, k = gate.shape
-            both = torch.stack([gate.view(ff // 16, 16, k), up.view(ff // 16, 16, k)], dim=1)
-            self.gate_up = Linear(both.reshape(2 * ff, k))
+            self.gate_up = Linear(interleaved_gate_up(gate, up))
         else:
             self.gate_up = Linear.stacked([gate, up])
         self.down = Linear(tensor_of(spec, "down", weights))
@@ -78,9 +89,11 @@ class NoFeedForward:
 
 class GatedFeedForward:
     """``y = W_down (act(W_gate h + b_gate) * (W_up h + b_up)) + b_down`` with ``activation``
-    ``silu`` or ``gelu_tanh`` (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))); the biases
-    (tensor roles ``gate_bias``, ``up_bias``, ``down_bias``) are optional.  Without biases and
-    with silu it is the standard part and runs on its fused product."""
+    ``silu`` or ``gelu_tanh`` (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))), or in the form
+    ``clamped_swish`` with ``limit`` L: ``g sigmoid(1.702 g) (u + 1)``, the gate g bounded above by L
+    and the other half u to -L .. L.  The biases (tensor roles ``gate_bias``, ``up_bias``,
+    ``down_bias``) are optional.  Without biases and with silu it is the standard part and runs on
+    its fused product; the clamped form without biases is fused into its product too."""
 
     graph_safe = True
 
@@ -99,8 +112,12 @@ class GatedFeedForward:
         if self.activation == "silu" and all(v is None for v in b.values()):
             self.plain = SwiGLU(spec, weights, dtype, device)
             return
-        self.gate_up = Linear.stacked([tensor_of(spec, "gate", weights),
-                                       tensor_of(spec, "up", weights)])
+        gate, up = tensor_of(spec, "gate", weights), tensor_of(spec, "up", weights)
+        self.limit = float(spec.get("limit") or 0.0)
+        self.fused = (self.activation == "clamped_swish" and all(v is None for v in b.values())
+                      and kernels.gated_interleave_ok(gate, up))
+        self.gate_up = Linear(interleaved_gate_up(gate, up)) if self.fused \
+            else Linear.stacked([gate, up])
         self.gate_up_bias = None if b["gate"] is None else torch.cat(
             [b["gate"].to(torch.float32), b["up"].to(torch.float32)]).contiguous()
         self.down = Linear(tensor_of(spec, "down", weights), b["down"])
@@ -116,14 +133,19 @@ class GatedFeedForward:
             self.plain.forward(ctx, h, x, accumulate=accumulate)
             return
         rows = ctx.rows
+        act = ctx.buffer("ffn.act", (rows, self.ff))
+        if self.fused:
+            kernels.gate_up_clamped(h, self.gate_up.weight, act, self.limit)
+            self.down(act, x, accumulate=accumulate)
+            return
         # (few rows: the product adds partial sums into a buffer kept at zero, which the
         # activation kernel clears again)
         kept_zero = rows <= kernels.SPLIT_K_MAX_ROWS
         gu = ctx.buffer("ffn.gate_up.z" if kept_zero else "ffn.gate_up", (rows, 2 * self.ff),
                         torch.float32, zero=kept_zero)
         self.gate_up(h, gu, out_is_zero=kept_zero)
-        act = ctx.buffer("ffn.act", (rows, self.ff))
-        kernels.gated_act(gu, self.gate_up_bias, act, self.activation, clear=kept_zero)
+        kernels.gated_act(gu, self.gate_up_bias, act, self.activation, clear=kept_zero,
+                          limit=self.limit)
         self.down(act, x, accumulate=accumulate)
 
 
@@ -189,7 +211,13 @@ class RoutedExperts:
         corr = optional_tensor_of(spec, "correction", weights)
         self.correction = None if corr is None else \
             corr.to(device=router.device, dtype=torch.float32).contiguous()
-        if self.correction is not None and self.scores == "softmax_chosen":
+        self.weight_on = spec.get("weight_on", "output")
+        if self.weight_on not in ("output", "input"):
+            raise ConfigError(f"routed experts: weight_on '{self.weight_on}' (output or input)")
+        if self.weight_on == "input" and (self.activation != "clamped_swish" or self.identity):
+            raise ConfigError("routed experts: weights on the input are there for experts of the "
+                              "clamped form")
+        if self.correction is not None and self.scores in ("softmax_chosen", "sigmoid"):
             raise ConfigError("routed experts: a correction of the choice needs scores over "
                               "all router outputs")
         bias = optional_tensor_of(spec, "router_bias", weights)
@@ -197,18 +225,25 @@ class RoutedExperts:
             else bias.to(torch.float32)
         sg = optional_tensor_of(spec, "shared_gate", weights)
         self.shared = None
+        self.shared_gated = sg is not None
         if spec.get("shared") is not None:
-            if sg is None or tuple(sg.shape) != (1, W):
-                raise ConfigError("routed experts: a shared expert needs its gate [1, hidden]")
             self.shared = build_part("feed_forward", spec["shared"], weights, dtype, device)
-            router = torch.cat([router, sg.to(torch.float32)])
-            bias = torch.cat([bias, torch.zeros(1, device=bias.device)])
+            if sg is not None:
+                if tuple(sg.shape) != (1, W):
+                    raise ConfigError("routed experts: the shared expert's gate is [1, hidden]")
+                router = torch.cat([router, sg.to(torch.float32)])
+                bias = torch.cat([bias, torch.zeros(1, device=bias.device)])
         # the router (and the shared expert's gate as its last row) stays 32-bit
         self.router = Linear(router.contiguous(), bias)
+        self.interleaved = False
         if self.gated:
-            self.gate_up = torch.stack([torch.cat([tensor_of(spec, f"gate{e}", weights),
-                                                   tensor_of(spec, f"up{e}", weights)])
-                                        for e in range(E)]).contiguous()           # [E, 2 ff, W]
+            gate = torch.stack([tensor_of(spec, f"gate{e}", weights) for e in range(E)])
+            up = torch.stack([tensor_of(spec, f"up{e}", weights) for e in range(E)])
+            # for the grouped product an expert's gate and up rows alternate in blocks of 16
+            self.interleaved = gate.is_cuda and kernels.moe_grouped_ok(gate.dtype, W, ff)
+            self.gate_up = interleaved_gate_up(gate, up) if self.interleaved \
+                else torch.cat([gate, up], dim=1).contiguous()                     # [E, 2 ff, W]
+            del gate, up
         else:       # (the name stays: without a gate it holds the up matrices alone, [E, ff, W])
             self.gate_up = torch.stack([tensor_of(spec, f"up{e}", weights)
                                         for e in range(E)]).contiguous()
@@ -240,7 +275,11 @@ class RoutedExperts:
         ident = h if self.identity else None
         shared = gate = None
         kept_zero = rows <= kernels.SPLIT_K_MAX_ROWS
-        if self.shared is not None:
+        if self.shared is not None and not self.shared_gated:
+            # without a gate the shared expert adds into the destination itself
+            self.shared.forward(ctx, h, x, accumulate=accumulate)
+            accumulate = True
+        elif self.shared is not None:
             # (few rows: the shared expert adds into a buffer kept at zero, cleared by the kernel
             # that sums the experts)
             shared = ctx.buffer("moe.shared.z" if kept_zero else "moe.shared", (rows, self.hidden),
@@ -256,27 +295,31 @@ class RoutedExperts:
             tile_group = ctx.buffer("moe.tiles", (tiles,), torch.int32)
             kernels.moe_align(ids, E, bn, pos, tile_group)
             xp = ctx.buffer("moe.x", (tiles * bn, self.hidden))
-            kernels.moe_gather(h, pos, xp, top, ids if self.identity else None, E)
+            scale = None
+            if self.weight_on == "input":     # the products of a row are scaled: they are linear
+                scale = ctx.buffer("moe.scale", (tiles * bn,), torch.float32)
+            kernels.moe_gather(h, pos, xp, top, ids if self.identity else None, E,
+                               wts if scale is not None else None, scale)
             act = ctx.buffer("moe.act", (tiles * bn, self.ff))
-            if self.activation == "silu":
-                kernels.gemm_grouped(xp, self.gate_up, act, tile_group, bn, gated=True)
-            elif not self.gated:
+            if self.gated:
+                kernels.gemm_grouped(xp, self.gate_up, act, tile_group, bn, gated=True,
+                                     interleaved=True, activation=self.activation,
+                                     limit=self.limit, row_scale=scale)
+            else:
                 u = ctx.buffer("moe.up", (tiles * bn, self.ff), torch.float32)
                 kernels.gemm_grouped(xp, self.gate_up, u, tile_group, bn, gated=False)
                 kernels.act_rows(u, act, self.activation)
-            else:       # the product as it is, then the activation over the padded buffer
-                gu = ctx.buffer("moe.gate_up", (tiles * bn, 2 * self.ff), torch.float32)
-                kernels.gemm_grouped(xp, self.gate_up, gu, tile_group, bn, gated=False)
-                kernels.gated_act(gu, None, act, self.activation, limit=self.limit)
             d = ctx.buffer("moe.down", (tiles * bn, self.hidden), torch.float32)
             kernels.gemm_grouped(act, self.down, d, tile_group, bn, gated=False)
-            kernels.moe_combine(d, pos, wts, x, accumulate, shared, gate, clear_shared=kept_zero,
+            kernels.moe_combine(d, pos, wts if scale is None else None, x, accumulate, shared, gate, clear_shared=kept_zero,
                                 ids=ids if self.identity else None, experts=E,
                                 identity_input=ident)
             return
         act = ctx.buffer("moe.act", (rows, top, self.ff))
-        kernels.moe_gate_up_rows(h, self.gate_up, ids, act, self.activation, self.limit)
-        kernels.moe_down_rows(act, self.down, ids, wts, x, accumulate, shared, gate,
+        on_input = self.weight_on == "input"
+        kernels.moe_gate_up_rows(h, self.gate_up, ids, act, self.activation, self.limit,
+                                 wts if on_input else None, self.interleaved)
+        kernels.moe_down_rows(act, self.down, ids, None if on_input else wts, x, accumulate, shared, gate,
                               clear_shared=kept_zero, identity_input=ident)
 
 

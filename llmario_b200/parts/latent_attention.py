@@ -8,7 +8,9 @@ With ``h`` the mixer's input, per token:
   numbers, not normed: one rotated key part shared by all heads];
 * head h's plain key is ``U_k,h c`` and its value ``U_v,h c``; the score of a query and a key is
   ``(q_plain . k_plain + q_rot . k_rot) * scale``;
-* the rotation turns adjacent pairs (2i, 2i + 1) of the rotated parts by ``pos * base^(-2i/dims)``;
+* the rotation turns pairs of the rotated parts by ``pos * base^(-2i/dims)``: adjacent ones
+  (2i, 2i + 1) for ``rope_normal``, (i, i + dims/2) for ``rope_neox`` (whose pairs are brought side by
+  side by ordering the projections' rows once: scores do not depend on the order of channels);
 * a query at position p sees the keys at p - window + 1 .. p; an optional ``sink`` per head adds
   ``exp(sink)`` to the softmax's sum (a key without a value);
 * the heads' outputs, concatenated, are projected by ``W_o``.
@@ -61,6 +63,13 @@ class LatentAttention:
         t = {r: tensor_of(spec, r, weights) for r in ("dq", "uq", "dkv", "uk", "uv", "o")}
         if tuple(t["dkv"].shape) != (C + R, self.hidden) or tuple(t["uq"].shape) != (H * (D + R), self.q_rank):
             raise ConfigError("latent attention: the projections do not have the sizes of the spec")
+        if self.position is not None and not hasattr(self.position, "head_permutation"):
+            rot = self.position.rot_dim
+            order = [j for i in range(rot // 2) for j in (i, i + rot // 2)] + list(range(rot, R))
+            order = torch.tensor(order, dtype=torch.long, device=t["uq"].device)
+            uq = t["uq"].view(H, D + R, self.q_rank)
+            t["uq"] = torch.cat([uq[:, :D], uq[:, D:][:, order]], dim=1).reshape(t["uq"].shape)
+            t["dkv"] = torch.cat([t["dkv"][:C], t["dkv"][C:][order]])
         self.down_proj = _padded_rows([t["dq"], t["dkv"]], self.hidden)   # [c_q | c | k_rot]
         self.q_proj = Linear(t["uq"])
         # head h's key map, transposed: it is applied to the query's plain part

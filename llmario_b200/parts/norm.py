@@ -1,5 +1,6 @@
 """RMS norm: ``y = x * 1/sqrt(mean(x^2) + eps) * w`` with sums and scale in 32-bit; the weight is
-the plain gain (crates/engine/cpu/src/ops.rs:18-29)."""
+the plain gain (crates/engine/cpu/src/ops.rs:18-29) or, with ``zero_centred``, what the gain has
+beyond one (``1 + w``, added once in 32-bit when the part is built)."""
 from __future__ import annotations
 
 from typing import Dict, Optional
@@ -19,6 +20,8 @@ class RmsNorm:
         self.eps = float(spec["eps"])
         self.weight = tensor_of(spec, "weight", weights).to(device=device, dtype=torch.float32)
         assert self.weight.numel() == self.width
+        if spec.get("zero_centred"):
+            self.weight = 1.0 + self.weight
 
     def apply(self, ctx: Optional[StepContext], x: torch.Tensor, out: torch.Tensor,
               rows_index: Optional[torch.Tensor] = None) -> None:
