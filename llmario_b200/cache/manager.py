@@ -51,13 +51,15 @@ class PagedKV:
     (None = all); with a window, the first ``keep_first`` keys are seen from everywhere and
     their pages never go back.  ``every`` > 1: one entry per so many tokens (entry b belongs to
     the tokens ``b * every ..``, written when the last of them has come), for layers that keep
-    a pooled key and value per block of tokens."""
+    a pooled key and value per block of tokens.  ``planes`` 1: only key rows are kept (a layer
+    whose values are a part of its keys)."""
 
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     keep_first: int = 0
     every: int = 1
+    planes: int = 2
 
 
 @dataclass(frozen=True)
@@ -162,7 +164,7 @@ class _Group:
     need: PagedKV
     n_pages: int
     entries: List[int] = field(default_factory=list)   # run-order entries stored here
-    storage: Optional[torch.Tensor] = None              # [page, slot, 2, Hkv, page_size, hd]
+    storage: Optional[torch.Tensor] = None         # [page, slot, planes, Hkv, page_size, hd]
     table: Optional[torch.Tensor] = None                # device int32 [requests, pages/request]
 
 
@@ -261,7 +263,7 @@ class CacheManager:
             n = g.need
             # per KV head the positions of a page lie one after the other: a kernel that serves
             # one KV head reads page_size * head_dim contiguous elements per page
-            g.storage = torch.zeros((g.n_pages, len(g.entries), 2, n.num_kv_heads,
+            g.storage = torch.zeros((g.n_pages, len(g.entries), n.planes, n.num_kv_heads,
                                      self.page_size, n.head_dim), dtype=dtype, device=device)
             g.table = torch.full((self.max_requests, self.pages_per_request), -1,
                                  dtype=torch.int32, device=device)
@@ -273,7 +275,7 @@ class CacheManager:
         size = torch.empty((), dtype=dtype).element_size()
         total = 0
         for g in self.groups:
-            total += (g.n_pages * len(g.entries) * 2 * self.page_size * g.need.num_kv_heads *
+            total += (g.n_pages * len(g.entries) * g.need.planes * self.page_size * g.need.num_kv_heads *
                       g.need.head_dim * size)
         return total
 
@@ -283,7 +285,7 @@ class CacheManager:
         gi, slot = self._where[entry]
         g = self.groups[gi]
         st = g.storage
-        return CacheView(st[0, slot, 0], st[0, slot, 1], st.stride(0), g.table, self.page_size,
+        return CacheView(st[0, slot, 0], st[0, slot, -1], st.stride(0), g.table, self.page_size,
                          gi, st, slot)
 
     def state_of(self, entry: int) -> Optional[torch.Tensor]:

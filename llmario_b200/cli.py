@@ -70,10 +70,16 @@ PAVATAR_PRESETS = {"pavatar-0.6b": ("qwen3-0.6b", 28), "pavatar-8b": ("qwen3-8b"
                    "pavatar-tiny": ("tiny-b", 4)}
 
 
+# Momuvik models of the same sizes (random weights): latent attention in every layer, the
+# feed-forwards repeating (dense, routed experts twice, dense).
+MOMUVIK_PRESETS = {"momuvik-0.6b": ("qwen3-0.6b", 28), "momuvik-8b": ("qwen3-8b", 36),
+                   "momuvik-tiny": ("tiny-b", 4)}
+
+
 def is_preset(name: str) -> bool:
     return name.lower() in PRESETS or name.lower() in VUNASUN_PRESETS \
         or name.lower() in RUNIDRA_PRESETS or name.lower() in PEMOLORN_PRESETS \
-        or name.lower() in PAVATAR_PRESETS
+        or name.lower() in PAVATAR_PRESETS or name.lower() in MOMUVIK_PRESETS
 
 
 def preset_config(name: str, num_layers: Optional[int] = None):
@@ -118,6 +124,16 @@ def preset_config(name: str, num_layers: Optional[int] = None):
                                   p["num_attention_heads"], p["num_key_value_heads"],
                                   p["head_dim"], int(num_layers or layers), p["vocab_size"],
                                   rank=8 if tiny else 64)
+
+    if name.lower() in MOMUVIK_PRESETS:
+        from .config.momuvik import sized_like as momuvik_sized_like
+
+        base, layers = MOMUVIK_PRESETS[name.lower()]
+        p = PRESETS[base]
+        small = {"kv_rank": 56, "rot": 16, "dim": 32} if base.startswith("tiny") else {}
+        return momuvik_sized_like(p["hidden_size"], p["intermediate_size"],
+                                  p["num_attention_heads"], int(num_layers or layers),
+                                  p["vocab_size"], **small)
 
     raw = dict(PRESETS[name.lower()], architectures=["Qwen3ForCausalLM"], model_type="qwen3")
     if num_layers:
@@ -291,7 +307,8 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
                                  "one B200: token ids in, token ids out")
     sub = ap.add_subparsers(dest="cmd", required=True)
     run = sub.add_parser("run", help="generate from a prompt of token ids")
-    run.add_argument("model", help="model folder, or a preset name: " + ", ".join(list(PRESETS) + list(VUNASUN_PRESETS) + list(RUNIDRA_PRESETS) + list(PEMOLORN_PRESETS) + list(PAVATAR_PRESETS)))
+    run.add_argument("model", help="model folder, or a preset name: " + ", ".join(list(PRESETS) + list(VUNASUN_PRESETS) + list(RUNIDRA_PRESETS) + list(PEMOLORN_PRESETS) + list(PAVATAR_PRESETS)
+                     + list(MOMUVIK_PRESETS)))
     run.add_argument("--tokens", default=None, help="comma-separated prompt token ids")
     run.add_argument("--prompt-len", type=int, default=16,
                      help="without --tokens: this many random ids")

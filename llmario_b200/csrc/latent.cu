@@ -12,7 +12,8 @@
 namespace {
 // One block per row.  proj[row] = [ query latent (q_rank) | key-value latent (kv_rank) | key part
 // to rotate (rot_dim) ].  The query latent is normed (gain wq) into cq_out; the key-value latent
-// is normed (gain wc) into the row's place in the K plane and, the same values, the V plane;
+// is normed (gain wc) into the row's place in the K plane and, the same values, the V plane (null:
+// the cache has none, values are read from the key rows);
 // the key part is rotated by the row's angles (cos_sin[row][i] = (cos, sin) of angle i, the first
 // rot_half pairs; null: no rotation) and written behind the latent in the K plane.  The V plane's
 // channels behind the latent are never written and stay zero.  clear_proj: the row of proj that
@@ -54,7 +55,7 @@ __global__ void __launch_bounds__(128) latent_store_kernel(
   for (int i = tid; i < kv_rank; i += blockDim.x) {
     const T v = from_f32<T>(c[i] * sc * wc[i]);
     k_plane[off + i] = v;
-    v_plane[off + i] = v;
+    if (v_plane) v_plane[off + i] = v;
   }
   const float* kr = c + kv_rank;
   for (int j = tid; j < rot_dim; j += blockDim.x) {

@@ -121,6 +121,12 @@ int llm_attention_tcgen05_x2(const void* q, void* out, int rows, const void* k_c
                              long long page_stride, long long n_pages, const int* block_table,
                              int table_stride, const int* items, int n_items, int Hq, int Hkv, int hd,
                              int page_size, float scale, int window, int* status, cudaStream_t stream);
+int llm_attention_latent_ok(int kd, int vdim, int page_size);
+int llm_attention_latent(const void* q, void* out, int flat_rows, int H, int kd, int vdim, const void* k_cache,
+                         long long page_stride, long long n_pages, const int* block_table, int table_stride,
+                         const int* items, int n_items, const int* row_pos, const int* row_slot, int page_size,
+                         float scale, int window, int splits, float* part_o, float* part_ml, const float* sink,
+                         int* status, cudaStream_t stream);
 }
 
 namespace {
@@ -142,6 +148,8 @@ constexpr int PERSISTENT_ATTENTION_MAX_KEYS = 6144;
 // gathered into scratch pages of GATHER_PAGE positions when the portion has at least
 // GATHER_MIN_PAIRS (token, head of the group) pairs.  (The tcgen05 kernel reaches about twice the
 // rate with TMA boxes; the copy costs about as much as the attention of 90 / group tokens.)
+constexpr int LATENT_ROWS = 128;            // flat (token, head) rows of a CTA of attention_latent.cu
+constexpr int LATENT_TILE = 64;             // and the keys of its tiles
 constexpr int GATHER_PAGE = 128;
 constexpr int GATHER_MIN_PAIRS = 512;
 int g_gather = 1;                           // 0: never gather (for measurements)
@@ -165,7 +173,7 @@ int g_fuse_mode = 0;                        // 0: when few waves, 1: always, 2: 
 enum Kind : int {
   K_NORM, K_GEMM_TCGEN05, K_GEMM_SIMT, K_ROPE_TABLE, K_ROPE_STORE, K_DECODE_FUSED, K_DECODE_TMA, K_DECODE,
   K_FLASH, K_MERGE, K_TCGEN05, K_TCGEN05_X2, K_GENERIC, K_SILU_MUL, K_KV_GATHER, K_DECODE_PERSISTENT,
-  K_EXTRAS, N_KINDS
+  K_EXTRAS, K_LATENT, N_KINDS
 };
 long long g_counts[N_KINDS] = {};
 
@@ -301,6 +309,12 @@ struct GatherPlan {
   const int* direct = nullptr;      // device: items read from the cache itself
 };
 
+// The step's (token, head) pairs as groups of up to LATENT_ROWS, for attention over latents.
+struct LatentPlan {
+  int heads = 0, n = 0;
+  const int* items = nullptr;       // device quadruples (first flat row, flat rows, slot, 0)
+};
+
 // What is made once per step and shared by its layers (and by calls that come one by one from
 // Python parts): work items and the tables of cosines and sines.  Keyed by the step's id.
 struct StepCache {
@@ -308,6 +322,7 @@ struct StepCache {
   int uploads = 0;
   std::deque<Plan> plans;
   std::deque<GatherPlan> gathers;
+  std::deque<LatentPlan> latents;
   std::map<const float*, float*> rope;     // inv_freq table -> cos/sin of this step's rows
 };
 
@@ -319,6 +334,7 @@ StepCache& step_cache(long long step_id) {
   if (c.step_id != step_id || step_id < 0) {
     c.plans.clear();
     c.gathers.clear();
+    c.latents.clear();
     c.rope.clear();
     c.uploads = 0;
     c.step_id = step_id;
@@ -333,11 +349,12 @@ struct Run {
   int launches = 0;
   std::deque<Plan>& plans;
   std::deque<GatherPlan>& gathers;
+  std::deque<LatentPlan>& latents;
   std::map<const float*, float*>& rope;
   int& uploads;
 
   Run(const LlmStepDesc& s, cudaStream_t str, StepCache& c)
-      : st(s), stream(str), ar(arena()), plans(c.plans), gathers(c.gathers), rope(c.rope), uploads(c.uploads) {}
+      : st(s), stream(str), ar(arena()), plans(c.plans), gathers(c.gathers), latents(c.latents), rope(c.rope), uploads(c.uploads) {}
 
   int check(int rc, Kind kind) {
     if (rc == 0) {
@@ -526,6 +543,61 @@ struct Run {
     *part_o = (float*)o;
     *part_ml = (float*)ml;
     return 0;
+  }
+
+  int latent_plan(int H, const LatentPlan** out) {
+    for (const LatentPlan& p : latents)
+      if (p.heads == H) { *out = &p; return 0; }
+    LatentPlan p;
+    p.heads = H;
+    std::vector<int> items;
+    for (int s = 0; s < st.n_segments; ++s) {
+      const int* g = st.segments + 4 * s;   // (first row, rows, slot, first position)
+      const int first = g[0] * H, n = g[1] * H;
+      for (int at = 0; at < n; at += LATENT_ROWS)
+        items.insert(items.end(), {first + at, n - at < LATENT_ROWS ? n - at : LATENT_ROWS, g[2], 0});
+    }
+    p.n = (int)items.size() / 4;
+    int* dev = nullptr;
+    int rc = ar.upload(items, uploads++, &dev, stream);
+    if (rc) return rc;
+    p.items = dev;
+    latents.push_back(p);
+    *out = &latents.back();
+    return 0;
+  }
+
+  // Attention over latents (attention_latent.cu): one key head whose values are the first value_dim
+  // channels of its key rows.  The keys are cut into parts when the step has few rows.
+  int latent_attention(const LlmLayerDesc& L, const LlmCallDesc& c, const void* q, void* out) {
+    const int H = L.num_heads, kd = L.head_dim, vd = L.value_dim > 0 ? L.value_dim : kd;
+    const int chunks = llm_attention_latent_ok(kd, vd, c.page_size);
+    if (!chunks || st.dtype != LLM_BF16 || c.n_pages <= 0) return LLM_ERR_UNSUPPORTED;
+    const int* items = nullptr;
+    int n = st.rows, groups = st.rows * ceil_div(H, LATENT_ROWS);
+    if (!st.all_single) {
+      const LatentPlan* plan = nullptr;
+      const int rc = latent_plan(H, &plan);
+      if (rc) return rc;
+      items = plan->items, n = groups = plan->n;
+    }
+    int splits = 1;
+    if ((long long)groups * chunks < sm_count())
+      splits = llm_decode_splits(groups, chunks, reach_of(L.window, st.max_pos), sm_count(), LATENT_TILE);
+    float *part_o = nullptr, *part_ml = nullptr;
+    if (splits > 1) {
+      void *o = nullptr, *ml = nullptr;
+      int rc = buffer(B_PART_O, (size_t)st.rows * H * splits * vd * sizeof(float), &o);
+      if (rc) return rc;
+      rc = buffer(B_PART_ML, (size_t)st.rows * H * splits * chunks * 2 * sizeof(float), &ml);
+      if (rc) return rc;
+      part_o = (float*)o, part_ml = (float*)ml;
+    }
+    const int rc = check(llm_attention_latent(q, out, st.rows * H, H, kd, vd, c.k, c.page_stride, c.n_pages, c.block_table,
+                                              c.table_stride, items, n, st.row_pos, st.row_slot, c.page_size, L.scale,
+                                              L.window, splits, part_o, part_ml, L.sink, st.status, stream), K_LATENT);
+    if (rc == 0 && splits > 1) ++launches, ++g_counts[K_MERGE];
+    return rc;
   }
 
   // causal attention of every row over its own request's cached keys (kernels.attention)
@@ -847,6 +919,19 @@ LLM_EXPORT int llm_attention_step(const LlmLayerDesc* layer, const LlmCallDesc* 
   if (!step->all_single && (step->segments == nullptr || step->n_segments <= 0)) return LLM_ERR_ARGUMENT;
   Run run(*step, stream, step_cache(step->step_id));
   const int rc = run.attention(*layer, *call, q, out);
+  if (n_launches) *n_launches = run.launches;
+  return rc;
+}
+
+// The same for attention over latents: one key head, values the first value_dim channels of the key
+// rows (call->v is not read; call->n_pages says how many pages there are).
+LLM_EXPORT int llm_latent_attention_step(const LlmLayerDesc* layer, const LlmCallDesc* call, const LlmStepDesc* step,
+                                         const void* q, void* out, int* n_launches, cudaStream_t stream) {
+  if (n_launches) *n_launches = 0;
+  if (step->rows <= 0) return 0;
+  if (!step->all_single && (step->segments == nullptr || step->n_segments <= 0)) return LLM_ERR_ARGUMENT;
+  Run run(*step, stream, step_cache(step->step_id));
+  const int rc = run.latent_attention(*layer, *call, q, out);
   if (n_launches) *n_launches = run.launches;
   return rc;
 }

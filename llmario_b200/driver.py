@@ -73,6 +73,8 @@ def _lib():
         l.llm_attention_step.argtypes = [POINTER(LayerDesc), POINTER(CallDesc), POINTER(StepDesc),
                                          c_void_p, c_void_p, POINTER(c_int), c_void_p]
         l.llm_attention_step.restype = c_int
+        l.llm_latent_attention_step.argtypes = l.llm_attention_step.argtypes
+        l.llm_latent_attention_step.restype = c_int
         l.llm_set_gather.argtypes = [c_int]
         l.llm_set_gather.restype = None
         _declared = True
@@ -93,7 +95,7 @@ def arena_drop() -> None:
 
 KINDS = ("norm", "gemm_tcgen05", "gemm_simt", "rope_table", "rope_store", "decode_fused",
          "decode_tma", "decode", "flash", "merge", "tcgen05", "tcgen05_x2", "generic", "silu_mul",
-         "kv_gather", "decode_persistent", "outside_window")
+         "kv_gather", "decode_persistent", "outside_window", "latent")
 
 
 def kernel_counts() -> Dict[str, int]:
@@ -152,7 +154,7 @@ def fill_call(c: CallDesc, layer: int, writes_cache: bool, view) -> None:
     c.page_stride = view.page_stride
     c.k, c.v, c.block_table = view.k.data_ptr(), view.v.data_ptr(), view.block_table.data_ptr()
     st = getattr(view, "storage", None)
-    if st is not None and st.is_contiguous() and st.dim() == 6:
+    if st is not None and st.is_contiguous() and st.dim() == 6 and st.shape[2] == 2:
         c.storage, c.n_pages, c.n_slots, c.slot = st.data_ptr(), st.shape[0], st.shape[1], view.slot
     else:
         c.storage, c.n_pages, c.n_slots, c.slot = None, 0, 0, 0
@@ -198,6 +200,35 @@ def tensor_core_attention(dtype: torch.dtype, view, num_heads: int, num_kv_heads
     group = num_heads // num_kv_heads
     return (dtype == torch.bfloat16 and head_dim in (64, 128) and group <= 16 and 128 % group == 0
             and (view.page_stride * 2) % 16 == 0)
+
+
+def latent_attention(ctx, q: torch.Tensor, out: torch.Tensor, view, num_heads: int, key_dim: int,
+                     value_dim: int, scale: float, window: Optional[int],
+                     sink: Optional[torch.Tensor] = None) -> None:
+    """Causal attention of every row and head of the step over one shared key row per token, whose
+    first ``value_dim`` channels are the value, on the tensor cores (``csrc/attention_latent.cu``;
+    sizes it takes: :func:`kernels.attention_latent_ok`).  q ``[rows, heads * key_dim]``, out
+    ``[rows, heads * value_dim]``, bfloat16; ``window`` and ``sink`` as in :func:`attention`."""
+    kernels._cuda(q, out, view.k, view.block_table, sink)
+    assert q.dtype == out.dtype == torch.bfloat16 and q.is_contiguous() and out.is_contiguous()
+    assert q.numel() == ctx.rows * num_heads * key_dim
+    assert out.numel() == ctx.rows * num_heads * value_dim
+    assert sink is None or (sink.dtype == torch.float32 and sink.numel() == num_heads)
+    layer = LayerDesc()
+    layer.num_heads, layer.num_kv_heads, layer.head_dim = num_heads, 1, key_dim
+    layer.scale, layer.window, layer.value_dim = scale, int(window or 0), value_dim
+    if sink is not None:
+        layer.sink = sink.data_ptr()
+    call = CallDesc()
+    fill_call(call, 0, True, view)
+    call.n_pages = view.storage.shape[0]
+    rc = _lib().llm_latent_attention_step(ctypes.byref(layer), ctypes.byref(call),
+                                          ctypes.byref(describe_step(ctx)), q.data_ptr(),
+                                          out.data_ptr(), ctypes.byref(_launches),
+                                          kernels._stream())
+    kernels.launches += _launches.value
+    if rc != 0:
+        kernels._check(rc, f"latent attention (key row of {key_dim}, values of {value_dim})")
 
 
 def attention(ctx, q: torch.Tensor, out: torch.Tensor, view, num_heads: int, num_kv_heads: int,

@@ -55,6 +55,9 @@ def _signatures():
         "llm_attention_generic": [P, P, P, P, I, L, P, I, P, P, I, I, I, I, I, F, I, P, I, P],
         "llm_attention_generic_ext": [P, P, P, P, I, L, P, I, P, P, I, I, I, I, I, F, I, P, I, I, P,
                                       P, L, P, I, I, P],
+        "llm_attention_latent_ok": [I, I, I],
+        "llm_attention_latent": [P, P, I, I, I, I, P, L, L, P, I, P, I, P, P, I, F, I, I, P, P, P, P,
+                                 P],
         "llm_qkv_store": [P, I, P, I, P, I, P, P, P, P, P, P, I, L, P, I, P, P, I, I, I, I, I, I, I,
                           I, F, I, I, P],
         "llm_pool_blocks": [P, P, L, P, I, P, P, L, P, I, P, P, I, I, I, I, I, I, P],
@@ -1404,14 +1407,15 @@ def latent_store(proj: torch.Tensor, q_weight: torch.Tensor, c_weight: torch.Ten
                  rot_dim: int, eps: float, write_cache: bool = True, clear: bool = False) -> None:
     """From proj (float32 [rows, >= q_rank + kv_rank + rot_dim]): the normed query latent into
     ``cq_out`` and the key row [normed latent | rotated key part] into the paged cache ``view``
-    (K plane whole, V plane the latent alone).  ``cos_sin``: float32 [rows, pairs, 2]."""
+    (K plane whole; V plane, where the cache has one, the latent alone).  ``cos_sin``: float32 [rows, pairs, 2]."""
     _cuda(proj, q_weight, c_weight, cos_sin, cq_out, view.k, view.v, row_slot, row_pos)
     rows = cq_out.shape[0]
     assert proj.dtype == torch.float32 and proj.stride(1) == 1 and cq_out.is_contiguous()
     assert cq_out.dtype == view.k.dtype and cq_out.shape[1] == q_rank
     half = 0 if cos_sin is None else cos_sin.shape[1]
     _check(lib().llm_latent_store(_ptr(proj), proj.stride(0), _ptr(q_weight), _ptr(c_weight),
-                                  _ptr(cos_sin), half, _ptr(cq_out), _ptr(view.k), _ptr(view.v),
+                                  _ptr(cos_sin), half, _ptr(cq_out), _ptr(view.k),
+                                  _ptr(view.v) if view.v.data_ptr() != view.k.data_ptr() else None,
                                   _dt(cq_out), view.page_stride, _ptr(view.block_table),
                                   view.block_table.stride(0), _ptr(row_slot), _ptr(row_pos), rows,
                                   view.page_size, q_rank, kv_rank, rot_dim, float(eps),
@@ -1432,6 +1436,14 @@ def latent_query(q: torch.Tensor, cos_sin: Optional[torch.Tensor], q_plain: torc
     _check(lib().llm_latent_query(_ptr(q), q.stride(0), _ptr(cos_sin), half, _ptr(q_plain),
                                   _ptr(q_full), _dt(q_full), rows, heads, dim, rot_dim, kv_rank,
                                   int(clear), _stream()), "latent_query")
+
+
+def attention_latent_ok(dtype: torch.dtype, key_dim: int, value_dim: int, page_size: int) -> bool:
+    """Whether the tensor-core kernel for attention over latents takes these sizes: bfloat16, key
+    rows of whole 16-byte units that fit a CTA's shared memory (up to about 700 channels), pages
+    of a multiple of 64 or of 8, 16 or 32 positions."""
+    return dtype == torch.bfloat16 and lib().llm_attention_latent_ok(key_dim, value_dim,
+                                                                     page_size) > 0
 
 
 HEAD_LINEAR_SIMT_ROWS = 128     # up to so many rows the per-head maps are one CUDA-core launch

@@ -19,6 +19,11 @@ The cache holds ``c`` and the rotated key part, nothing per head: one key row of
 rot_dim`` channels per token.  The heads' key maps are applied to the queries (``U_k,h^T q_plain``) and their value maps
 to the attention's output (``U_v,h sum_j p_j c_j``), so the attention itself runs as one shared key
 head whose values are the first ``kv_rank`` channels of its keys.
+
+Which kernels run it: key rows of 64 or 128 channels with up to 16 heads that divide 128 go to the
+kernels of ordinary attention (in bfloat16), which want a value row beside every key row; every
+other size keeps key rows alone and goes to the kernel for attention over latents (bfloat16) or to
+the generic one (32-bit, rows that are not whole 16-byte units, pages it does not take).
 """
 from __future__ import annotations
 
@@ -78,11 +83,14 @@ class LatentAttention:
         self.o_proj = Linear(t["o"])
         self.q_gain = _f32(tensor_of(spec, "dq_norm", weights), device)
         self.c_gain = _f32(tensor_of(spec, "dkv_norm", weights), device)
+        # the kernels of ordinary attention read value rows; the others find them in the key rows
+        self.value_rows = dtype == torch.bfloat16 and self.key_dim in (64, 128) and H <= 16 \
+            and 128 % H == 0
         sink = optional_tensor_of(spec, "sink", weights)
         self.sink = None if sink is None else _f32(sink, device)
 
     def cache_need(self):
-        return PagedKV(1, self.key_dim, self.window)
+        return PagedKV(1, self.key_dim, self.window, planes=2 if self.value_rows else 1)
 
     def streamed_weights(self):
         return [self.down_proj.weight, self.q_proj.weight, self.key_maps, self.value_maps,
@@ -114,14 +122,20 @@ class LatentAttention:
         kernels.latent_query(q, angles, q_plain, q_full, H, D, R, C, clear=kept_zero)
         kernels.head_linear(q_plain.view(rows, H, D), self.key_maps,
                             q_full.view(rows, H, self.key_dim)[:, :, :C])
-        # sum_j p_j c_j per head.  The tensor-core kernels work on whole value rows (what lies
-        # behind the latent in a value row of the cache is zero and never written); the generic
-        # kernel is told to stop at the latent's end.
-        whole = driver.tensor_core_attention(ctx.dtype, view, H, 1, self.key_dim)
+        # sum_j p_j c_j per head.  The kernels of ordinary attention work on whole value rows (what
+        # lies behind the latent in a value row of the cache is zero and never written); the
+        # others stop at the latent's end.
+        whole = self.value_rows and driver.tensor_core_attention(ctx.dtype, view, H, 1,
+                                                                 self.key_dim)
         vd = self.key_dim if whole else C
         mixed = ctx.buffer("latent.mixed", (rows, H * vd))
-        driver.attention(ctx, q_full, mixed, view, H, 1, self.key_dim, self.scale, self.mask,
-                         sink=self.sink, value_dim=None if whole else C)
+        if not self.value_rows and kernels.attention_latent_ok(ctx.dtype, self.key_dim, C,
+                                                               view.page_size):
+            driver.latent_attention(ctx, q_full, mixed, view, H, self.key_dim, C, self.scale,
+                                    self.mask, sink=self.sink)
+        else:
+            driver.attention(ctx, q_full, mixed, view, H, 1, self.key_dim, self.scale, self.mask,
+                             sink=self.sink, value_dim=None if whole else C)
         out = ctx.buffer("latent.out", (rows, H * V))
         kernels.head_linear(mixed.view(rows, H, vd)[:, :, :C], self.value_maps,
                             out.view(rows, H, V))

@@ -15,7 +15,7 @@ SLOPE = 1.702          # of the clamped gate's sigmoid
 
 
 def sigmoid(z):
-    return 1.0 / (1.0 + np.exp(-z))
+    return np.exp(-np.logaddexp(0.0, -np.asarray(z, F)))
 
 
 def unit_rms(x, eps):
