@@ -4,11 +4,14 @@
 // With one key head every (token, query head) pair of a request is one more row of the same
 // problem, so the queries are taken as a matrix of flat rows [tokens * heads][key channels] and a
 // CTA takes up to 128 consecutive ones, whatever the number of heads, one TMEM lane each.  A row's
-// position is that of its token.  Keys are walked in tiles of 64 aligned to absolute positions.
+// position is that of its token.  The product takes 128 rows whatever a CTA has; where it has
+// fewer (steps of single tokens), only
+// theirs are kept in shared memory and the product's other rows read what lies behind them: their
+// results are not used.  Keys are walked in tiles of 64 aligned to absolute positions.
 // Channels are cut into blocks of 64 (128 bytes, one swizzle span; the last block is filled with
 // zeros).  A tile's blocks that are also values of this CTA ("value blocks", at most four: 256
 // accumulator columns) stay in shared memory until the second product has read them; the other
-// blocks pass through a ring of their own and are free once the scores have read them.  With more
+// blocks pass, in groups, through a ring of their own and are free once the scores have read them.  With more
 // value blocks than a CTA takes, several CTAs share the same rows, each with its part of the value
 // channels; they make the scores anew.  The keys can be cut into `splits` parts whose results a merge
 // kernel joins (steps of few rows).
@@ -30,10 +33,9 @@
 namespace {
 
 constexpr int ROWS = 128;             // flat rows of a CTA (TMEM lanes)
+constexpr int MAX_VS = 4, MAX_XS = 8;  // most stages of value blocks, of groups of other blocks
 constexpr int KT = 64;                // keys per tile
-constexpr int QBLK = ROWS * 128;      // bytes of a block of 64 channels of the queries
-constexpr int KBLK = KT * 128;        // and of a tile's keys
-constexpr int MAX_VS = 4, MAX_XS = 8; // most stages of value blocks, of other blocks
+constexpr int KBLK = KT * 128;        // bytes of a block of 64 channels of a tile's keys
 constexpr int SMEM_LIMIT = 227 * 1024;
 
 struct Bars {
@@ -54,7 +56,8 @@ struct LatentArgs {
   const int* row_pos;
   const int* row_slot;
   long long rows_per_page;
-  int H, page_size, kd_blocks, vdim, v_blocks, chunks, vs, xs, tmem_cols;
+  int q_rows;                 // rows of queries in shared memory (a multiple of 8)
+  int H, page_size, kd_blocks, vdim, v_blocks, chunks, vs, xs, xg, tmem_cols;
   float scale_log2;
   int window, splits;
   bf16* out;                  // [flat rows][vdim]
@@ -73,10 +76,11 @@ __global__ void __launch_bounds__(224, 1) attention_latent_kernel(const __grid_c
   extern __shared__ uint8_t raw[];
   uint8_t* base_s = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
   const int nkb = a.kd_blocks;
-  uint8_t* q_s = base_s;                                     // [nkb][128 rows][128 bytes]
+  const uint32_t QBLK = (uint32_t)a.q_rows * 128;            // bytes of a block of 64 channels of the queries
+  uint8_t* q_s = base_s;                                     // [nkb][q_rows][128 bytes]
   uint8_t* v_s = q_s + (size_t)nkb * QBLK;                   // [vs][v_blocks][64 keys][128 bytes]
-  uint8_t* x_s = v_s + (size_t)a.vs * a.v_blocks * KBLK;     // [xs][64 keys][128 bytes]
-  Bars& sm = *reinterpret_cast<Bars*>(x_s + (size_t)a.xs * KBLK);
+  uint8_t* x_s = v_s + (size_t)a.vs * a.v_blocks * KBLK;     // [xs][xg][64 keys][128 bytes]
+  Bars& sm = *reinterpret_cast<Bars*>(x_s + (size_t)a.xs * a.xg * KBLK);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // the last items of a prompt have the most keys to walk: they are started first
   const int n_items = gridDim.x / a.chunks;
@@ -135,18 +139,32 @@ __global__ void __launch_bounds__(224, 1) attention_latent_kernel(const __grid_c
   }
   const int R = min(a.page_size, KT);
   const int* table = a.block_table + (size_t)slot * a.table_stride;
-  // one block of 64 channels of a tile's keys: a box per page that holds a key of the item
-  auto live_rows = [&](int base) {
-    int n = 0;
-    for (int p = base; p < base + KT; p += R) n += (p <= hi && p + R - 1 >= lo) ? R : 0;
-    return n;
-  };
-  auto load_block = [&](uint8_t* dst, int kb, int base, uint64_t* bar) {
-    for (int p = base; p < base + KT; p += R) {
-      if (p > hi || p + R - 1 < lo) continue;       // no key of the item here: the page may be gone
-      const long long row = (long long)table[p / a.page_size] * a.rows_per_page + p % a.page_size;
-      tma_load_2d(dst + (p - base) * 128, &map_k, kb * 64, (int)row, bar);
+  // Where a tile's keys lie: the row of the key matrix for each page it touches, -1 for a page without
+  // a key of the item (it may be gone).  Looked up a tile ahead of the loads that use it.
+  struct TileRows { int row[KT / 8]; int live; };
+  const int pieces = KT / R;
+  auto look_up = [&](int base, TileRows& t) {
+    t.live = 0;
+#pragma unroll
+    for (int g = 0; g < KT / 8; ++g) {
+      t.row[g] = -1;
+      const int p = base + g * R;
+      if (g < pieces && p <= hi && p + R - 1 >= lo) {
+        const int page = p / a.page_size;
+        t.row[g] = (int)((long long)table[page] * a.rows_per_page + (p - page * a.page_size));
+        t.live += R;
+      }
     }
+  };
+  // one block of 64 channels of a tile's keys: a box per page
+  auto load_block = [&](uint8_t* dst, int kb, const TileRows& t, uint64_t* bar) {
+    if (pieces == 1) {
+      tma_load_2d(dst, &map_k, kb * 64, t.row[0], bar);
+      return;
+    }
+#pragma unroll
+    for (int g = 0; g < KT / 8; ++g)
+      if (t.row[g] >= 0) tma_load_2d(dst + g * R * 128, &map_k, kb * 64, t.row[g], bar);
   };
 
   if (ntiles > 0) {
@@ -155,34 +173,46 @@ __global__ void __launch_bounds__(224, 1) attention_latent_kernel(const __grid_c
       mbar_expect_tx(&sm.q_full, (uint32_t)nkb * QBLK);
       for (int kb = 0; kb < nkb; ++kb) tma_load_2d(q_s + (size_t)kb * QBLK, &map_q, kb * 64, f0, &sm.q_full);
       bool ok = true;
-      long long n = 0;
-      for (int j = 0; j < ntiles && ok; ++j) {
-        const int base = (tile_first + j) * KT;
-        const uint32_t bytes = (uint32_t)live_rows(base) * 128;
-        for (int x = 0; x < nx; ++x, ++n) {
-          const int s = (int)(n % a.xs), kb = x < vb0 ? x : x + nv;
-          ok = mbar_wait(&sm.x_empty[s], (uint32_t)((n / a.xs) & 1) ^ 1);
+      int s = 0, n = 0;                 // the next stage of the ring; groups issued
+      uint32_t phase = 0;               // flips whenever the ring has gone round
+      TileRows now, next;
+      if (nx > 0) look_up(tile_first * KT, next);
+      for (int j = 0; j < ntiles && nx > 0 && ok; ++j) {
+        now = next;
+        const uint32_t bytes = (uint32_t)now.live * 128;
+        for (int x0 = 0; x0 < nx; x0 += a.xg) {
+          ok = mbar_wait(&sm.x_empty[s], phase ^ 1);
           if (!ok) { atomicExch(a.status, 5); *(volatile int*)&sm.dead = 1; break; }
-          mbar_expect_tx(&sm.x_full[s], bytes);
-          load_block(x_s + (size_t)s * KBLK, kb, base, &sm.x_full[s]);
+          const int g = min(a.xg, nx - x0);
+          mbar_expect_tx(&sm.x_full[s], bytes * g);
+          for (int x = x0; x < x0 + g; ++x)
+            load_block(x_s + (size_t)(s * a.xg + x - x0) * KBLK, x < vb0 ? x : x + nv, now, &sm.x_full[s]);
+          ++n;
+          if (++s == a.xs) s = 0, phase ^= 1;
         }
+        if (j + 1 < ntiles) look_up((tile_first + j + 1) * KT, next);
       }
       if (!ok) {     // let what is in flight land before the shared memory is given up
         mbar_wait(&sm.q_full, 0);
-        for (long long i = n > a.xs ? n - a.xs : 0; i < n; ++i)
+        for (int i = max(0, n - a.xs); i < n; ++i)
           mbar_wait(&sm.x_full[i % a.xs], (uint32_t)((i / a.xs) & 1));
       }
     } else if (warp == 6 && lane == 0) {
       // ---------------------------------------------------------------- value blocks
       bool ok = true;
-      int j = 0;
+      int j = 0, s = 0;
+      uint32_t phase = 0;
+      TileRows now, next;
+      look_up(tile_first * KT, next);
       for (; j < ntiles; ++j) {
-        const int s = j % a.vs, base = (tile_first + j) * KT;
-        ok = mbar_wait(&sm.v_empty[s], (uint32_t)((j / a.vs) & 1) ^ 1);
+        now = next;
+        ok = mbar_wait(&sm.v_empty[s], phase ^ 1);
         if (!ok) { atomicExch(a.status, 5); *(volatile int*)&sm.dead = 1; break; }
-        mbar_expect_tx(&sm.v_full[s], (uint32_t)(live_rows(base) * 128 * nv));
+        mbar_expect_tx(&sm.v_full[s], (uint32_t)(now.live * 128 * nv));
         for (int b = 0; b < nv; ++b)
-          load_block(v_s + (size_t)(s * a.v_blocks + b) * KBLK, vb0 + b, base, &sm.v_full[s]);
+          load_block(v_s + (size_t)(s * a.v_blocks + b) * KBLK, vb0 + b, now, &sm.v_full[s]);
+        if (++s == a.vs) s = 0, phase ^= 1;
+        if (j + 1 < ntiles) look_up((tile_first + j + 1) * KT, next);
       }
       if (!ok)
         for (int i = max(0, j - a.vs); i < j; ++i) mbar_wait(&sm.v_full[i % a.vs], (uint32_t)((i / a.vs) & 1));
@@ -192,45 +222,50 @@ __global__ void __launch_bounds__(224, 1) attention_latent_kernel(const __grid_c
                                ((uint32_t)(ROWS >> 4) << 24);
       bool ok = mbar_wait(&sm.q_full, 0);
       if (!ok) { atomicExch(a.status, 6); *(volatile int*)&sm.dead = 1; }
-      long long n = 0;
-      auto scores = [&](uint32_t acc, int kb, const uint8_t* blk, bool first) {
-        const uint32_t qa = smem_u32(q_s + (size_t)kb * QBLK), ka = smem_u32(blk);
+      int xstage = 0, vstage = 0, pstage = 0;          // stages of the rings: other blocks, values for S, for PV
+      uint32_t xphase = 0, vphase = 0;
+      const uint64_t q_desc = smem_desc(smem_u32(q_s));
+      const uint32_t x_addr = smem_u32(x_s), v_addr = smem_u32(v_s), v_stage = (uint32_t)a.v_blocks * KBLK;
+      auto scores = [&](uint32_t acc, int kb, uint32_t blk, bool first) {
+        const uint64_t qd = q_desc + (uint64_t)((uint32_t)kb * QBLK >> 4), kd = smem_desc(blk);
 #pragma unroll
         for (int ks = 0; ks < 4; ++ks)
-          tc_mma(acc, smem_desc(qa + ks * 32), smem_desc(ka + ks * 32), IDESC_S, (first && ks == 0) ? 0u : 1u);
+          tc_mma(acc, qd + (uint64_t)(ks * 2), kd + (uint64_t)(ks * 2), IDESC_S, (first && ks == 0) ? 0u : 1u);
       };
       for (int j = 0; j <= ntiles && ok; ++j) {
         if (j < ntiles) {
           const uint32_t acc = tmem + (uint32_t)(j & 1) * KT;
-          for (int x = 0; x < nx; ++x, ++n) {
-            const int s = (int)(n % a.xs);
-            ok = mbar_wait(&sm.x_full[s], (uint32_t)((n / a.xs) & 1));
+          for (int x0 = 0; x0 < nx; x0 += a.xg) {
+            ok = mbar_wait(&sm.x_full[xstage], xphase);
             if (!ok) break;
             tc_fence_after();
-            scores(acc, x < vb0 ? x : x + nv, x_s + (size_t)s * KBLK, x == 0);
-            tc_commit(&sm.x_empty[s]);
+            for (int x = x0; x < min(nx, x0 + a.xg); ++x)
+              scores(acc, x < vb0 ? x : x + nv, x_addr + (uint32_t)(xstage * a.xg + x - x0) * KBLK, x == 0);
+            tc_commit(&sm.x_empty[xstage]);
+            if (++xstage == a.xs) xstage = 0, xphase ^= 1;
           }
-          const int s = j % a.vs;
-          ok = ok && mbar_wait(&sm.v_full[s], (uint32_t)((j / a.vs) & 1));
+          ok = ok && mbar_wait(&sm.v_full[vstage], vphase);
           if (!ok) { atomicExch(a.status, 6); *(volatile int*)&sm.dead = 1; break; }
           tc_fence_after();
           for (int b = 0; b < nv; ++b)
-            scores(acc, vb0 + b, v_s + (size_t)(s * a.v_blocks + b) * KBLK, nx == 0 && b == 0);
+            scores(acc, vb0 + b, v_addr + (uint32_t)vstage * v_stage + (uint32_t)b * KBLK, nx == 0 && b == 0);
+          if (++vstage == a.vs) vstage = 0, vphase ^= 1;
           tc_commit(&sm.s_full[j & 1]);
         }
         if (j >= 1) {
-          const int i = j - 1, s = i % a.vs;
+          const int i = j - 1;
           ok = mbar_wait(&sm.p_full[i & 1], (uint32_t)((i >> 1) & 1));
           if (!ok) { atomicExch(a.status, 6); *(volatile int*)&sm.dead = 1; break; }
           tc_fence_after();
           const uint32_t p_addr = tmem + (uint32_t)(i & 1) * KT;       // P over the first KT / 2 columns
-          const uint32_t va = smem_u32(v_s + (size_t)s * a.v_blocks * KBLK);
+          const uint32_t va = v_addr + (uint32_t)pstage * v_stage;
 #pragma unroll
           for (int ks = 0; ks < KT / UMMA_K; ++ks)
             tc_mma_ts(tmem + O_COL, p_addr + (uint32_t)ks * (UMMA_K / 2), smem_desc_mn(va + (uint32_t)ks * UMMA_K * 128, KBLK),
                       idesc_o, (i > 0 || ks > 0) ? 1u : 0u);
-          tc_commit(&sm.v_empty[s]);
+          tc_commit(&sm.v_empty[pstage]);
           tc_commit(&sm.o_done);
+          if (++pstage == a.vs) pstage = 0;
         }
       }
     } else if (warp >= 2 && warp < 6) {
@@ -243,6 +278,7 @@ __global__ void __launch_bounds__(224, 1) attention_latent_kernel(const __grid_c
       const int tok = flat / a.H, head = flat - tok * a.H;
       const int rpos = a.row_pos[tok];
       const int rlo = first_key(rpos, a.window);
+      const bool warp_idle = q4 * 32 >= nf;
       float m_used = -INFINITY, l = 0.f;
       bool ok = true;
       for (int j = 0; j < ntiles; ++j) {
@@ -255,20 +291,33 @@ __global__ void __launch_bounds__(224, 1) attention_latent_kernel(const __grid_c
         asm volatile("bar.sync 1, 128;" ::: "memory");
         if (*(volatile int*)&sm.stop[b]) { ok = false; break; }
         tc_fence_after();
+        if (warp_idle) {       // no row of the item: what the products make of these lanes is not used
+          if (lane == 0) mbar_arrive(&sm.p_full[b]);
+          continue;
+        }
         const uint32_t s_addr = tmem + lane_base + (uint32_t)b * KT;
         const int base = (tile_first + j) * KT;
-        const int c_hi = rvalid ? min(KT - 1, rpos - base) : -1;
+        // (a lane without a row of the item takes the first row's place; its result is not written)
+        const int c_hi = min(KT - 1, rpos - base);
         const int c_lo = max(0, rlo - base);
         // a tile that every row of the CTA sees completely needs no per-key tests
-        const bool interior = nf >= ROWS && base + KT - 1 <= pos_first && base >= first_key(hi, a.window);
+        const bool interior = base + KT - 1 <= pos_first && base >= first_key(hi, a.window);
         uint32_t v[KT];
 #pragma unroll
         for (int c = 0; c < KT; c += 32) tmem_ld32(s_addr + c, v + c);
         tmem_ld_wait();
         if (!interior) {
 #pragma unroll
-          for (int i = 0; i < KT; ++i)
-            if (i < c_lo || i > c_hi) v[i] = 0xff800000u;      // -inf: the key is not visible
+          for (int c = 0; c < KT; c += 32) {
+            // a bit per column: those from c_lo on, up to c_hi
+            const int n_hi = c_hi + 1 - c, n_lo = c_lo - c;
+            const uint32_t up_to = n_hi <= 0 ? 0u : n_hi >= 32 ? ~0u : (1u << n_hi) - 1u;
+            const uint32_t below = n_lo <= 0 ? 0u : n_lo >= 32 ? ~0u : (1u << n_lo) - 1u;
+            const uint32_t seen = up_to & ~below;
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              if (!(seen & (1u << i))) v[c + i] = 0xff800000u;      // -inf: the key is not visible
+          }
         }
         float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -329,7 +378,7 @@ __global__ void __launch_bounds__(224, 1) attention_latent_kernel(const __grid_c
         __syncwarp();
         if (lane == 0) mbar_arrive(&sm.p_full[b]);
       }
-      if (ok) {
+      if (ok && !warp_idle) {
         bool done = mbar_wait(&sm.o_done, (uint32_t)((ntiles - 1) & 1));
         if (!done) { if (lane == 0) atomicExch(a.status, 7); }
         done = __all_sync(0xffffffffu, done);
@@ -455,36 +504,40 @@ __global__ void __launch_bounds__(128) attention_latent_merge_kernel(const float
 }
 
 // how the shared memory of a CTA is laid out for these sizes; false: they do not fit
-struct Layout { int kd_blocks, chunks, v_blocks, vs, xs, smem, tmem_cols; };
-bool layout_for(int kd, int vdim, Layout* L) {
+struct Layout { int kd_blocks, chunks, v_blocks, vs, xs, xg, smem, tmem_cols, q_rows; };
+bool layout_for(int kd, int vdim, int q_rows, Layout* L) {
+  const int QBLK = q_rows * 128;
   const int nkb = (kd + 63) / 64, ncb = (vdim + 63) / 64;
   const int room = SMEM_LIMIT - 1024 - (int)sizeof(Bars) - nkb * QBLK;
   for (int chunks = (ncb + 3) / 4; chunks <= ncb; ++chunks) {
     const int nv = (ncb + chunks - 1) / chunks;
     if ((ncb + nv - 1) / nv != chunks) continue;       // (an empty last chunk)
-    // a CTA whose value blocks are fewer than nv has more of the others: there must be a ring
-    const bool others = nkb > nv || chunks > 1;
-    int vs = 2, xs = others ? 2 : 1;
+    // blocks of a CTA that are no values (the last CTA may have fewer value blocks than the others)
+    const int others = nkb - (ncb - (chunks - 1) * nv);
+    int vs = 2, xs = others ? 2 : 1, xg = 1;
     if ((vs * nv + xs) * KBLK > room) continue;
-    while (others && xs < 4 && xs < nkb && (vs * nv + xs + 1) * KBLK <= room) ++xs;
-    while (vs < MAX_VS && ((vs + 1) * nv + xs) * KBLK <= room) ++vs;
-    while (others && xs < MAX_XS && (vs * nv + xs + 1) * KBLK <= room) ++xs;
-    *L = Layout{nkb, chunks, nv, vs, xs, nkb * QBLK + (vs * nv + xs) * KBLK + (int)sizeof(Bars) + 1024,
-                nv <= 2 ? 256 : 512};
+    // as few groups as two stages of them fit: every group costs the issuing thread a wait
+    while (xg < others && (vs * nv + xs * (xg + 1)) * KBLK <= room) ++xg;
+    if (others) xg = (others + (others + xg - 1) / xg - 1) / ((others + xg - 1) / xg);
+    while (others && xs < 3 && (vs * nv + (xs + 1) * xg) * KBLK <= room) ++xs;
+    while (vs < MAX_VS && ((vs + 1) * nv + xs * xg) * KBLK <= room) ++vs;
+    while (others && xs < MAX_XS && (vs * nv + (xs + 1) * xg) * KBLK <= room) ++xs;
+    *L = Layout{nkb, chunks, nv, vs, xs, xg, nkb * QBLK + (vs * nv + xs * xg) * KBLK + (int)sizeof(Bars) + 1024,
+                nv <= 2 ? 256 : 512, q_rows};
     return true;
   }
   return false;
 }
+
 }  // namespace
 
 // Whether llm_attention_latent takes these sizes: returns the number of CTAs that share a group of
-// 128 flat rows (parts of the value channels), or 0.  page_size: a multiple of 64, or a power of
-// two of 8 to 32 positions.
+// 128 flat rows (parts of the value channels), or 0.  page_size: a multiple of 64, or 8, 16 or
+// 32 positions.
 LLM_EXPORT int llm_attention_latent_ok(int kd, int vdim, int page_size) {
   Layout L;
   if (kd <= 0 || kd % 8 || vdim <= 0 || vdim > kd) return 0;
-  if (page_size < 8 || (page_size < KT ? KT % page_size : page_size % KT)) return 0;
-  return layout_for(kd, vdim, &L) ? L.chunks : 0;
+  return page_size >= 8 && (page_size < KT ? KT % page_size == 0 : page_size % KT == 0) && layout_for(kd, vdim, ROWS, &L) ? L.chunks : 0;
 }
 
 // q [flat_rows][kd] and out [flat_rows][vdim] bfloat16, flat row = token * H + head; k_cache: this
@@ -509,16 +562,22 @@ LLM_EXPORT int llm_attention_latent(const void* q, void* out, int flat_rows, int
   const long long key_rows = (n_pages - 1) * rows_per_page + page_size;
   if (n_pages <= 0 || key_rows >= (1LL << 31)) return LLM_ERR_UNSUPPORTED;
   Layout L;
-  layout_for(kd, vdim, &L);
+  if (!layout_for(kd, vdim, ROWS, &L)) return LLM_ERR_UNSUPPORTED;
+  {      // (the part of the value channels a CTA takes stays that of full groups of rows)
+    const int q_rows = items || H >= ROWS ? ROWS : (H + 7) / 8 * 8;
+    Layout M;
+    if (layout_for(kd, vdim, q_rows, &M) && M.chunks == L.chunks) L = M;
+  }
   CUtensorMap mq, mk;
-  if (!llm_tensor_map(q, flat_rows, kd, kd, ROWS, 64, 0, &mq)) return LLM_ERR_UNSUPPORTED;
+  if (!llm_tensor_map(q, flat_rows, kd, kd, L.q_rows, 64, 0, &mq)) return LLM_ERR_UNSUPPORTED;
   if (!llm_tensor_map(k_cache, key_rows, kd, kd, page_size < KT ? page_size : KT, 64, 0, &mk)) return LLM_ERR_UNSUPPORTED;
   LatentArgs a;
   a.block_table = block_table, a.table_stride = table_stride, a.items = items;
   a.per_row = (H + ROWS - 1) / ROWS;
+  a.q_rows = L.q_rows;
   a.row_pos = row_pos, a.row_slot = row_slot, a.rows_per_page = rows_per_page;
   a.H = H, a.page_size = page_size, a.kd_blocks = L.kd_blocks, a.vdim = vdim, a.v_blocks = L.v_blocks;
-  a.chunks = L.chunks, a.vs = L.vs, a.xs = L.xs, a.tmem_cols = L.tmem_cols;
+  a.chunks = L.chunks, a.vs = L.vs, a.xs = L.xs, a.xg = L.xg, a.tmem_cols = L.tmem_cols;
   a.scale_log2 = scale * 1.4426950408889634f, a.window = window, a.splits = splits;
   a.out = (bf16*)out, a.part_o = part_o, a.part_ml = part_ml, a.sink = sink, a.status = status;
   static bool configured = false;

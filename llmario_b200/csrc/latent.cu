@@ -117,6 +117,53 @@ __global__ void latent_query_kernel(float* __restrict__ q, int q_stride, const f
     }
   }
 }
+// The same with four channels per thread and accesses of 16 and 8 bytes: dim, rot_dim, kv_rank and
+// the row stride multiples of four, every base aligned.
+template <typename T> __device__ __forceinline__ void put4(T* dst, float a, float b, float c, float d);
+template <> __device__ __forceinline__ void put4<float>(float* dst, float a, float b, float c, float d) {
+  *reinterpret_cast<float4*>(dst) = make_float4(a, b, c, d);
+}
+template <> __device__ __forceinline__ void put4<bf16>(bf16* dst, float a, float b, float c, float d) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
+  *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+}
+template <typename T>
+__global__ void __launch_bounds__(256) latent_query_vec_kernel(float* __restrict__ q, int q_stride,
+                                                               const float2* __restrict__ cos_sin, int rot_half,
+                                                               T* __restrict__ q_plain, T* __restrict__ q_full,
+                                                               unsigned total, int H, int dim, int rot_dim,
+                                                               int kv_rank, int clear) {
+  pdl_trigger();
+  pdl_wait();
+  const unsigned per_head = (unsigned)(dim + rot_dim) >> 2;
+  const int hd = kv_rank + rot_dim;
+  for (unsigned idx = blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += gridDim.x * blockDim.x) {
+    const unsigned rh = idx / per_head;
+    const int e = (int)(idx - rh * per_head) * 4;
+    const unsigned r = rh / (unsigned)H, h = rh - r * H;
+    float4* src = reinterpret_cast<float4*>(q + (size_t)r * q_stride + (size_t)h * (dim + rot_dim) + e);
+    float4 v = *src;
+    if (clear) *src = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (e < dim) {
+      put4<T>(q_plain + (size_t)rh * dim + e, v.x, v.y, v.z, v.w);
+      continue;
+    }
+    const int j = e - dim, i = j >> 1;
+    if (cos_sin) {
+      if (i < rot_half) {
+        const float2 cs = cos_sin[(size_t)r * rot_half + i];
+        const float a = v.x, b = v.y;
+        v.x = fmaf(a, cs.x, -b * cs.y), v.y = fmaf(b, cs.x, a * cs.y);
+      }
+      if (i + 1 < rot_half) {
+        const float2 cs = cos_sin[(size_t)r * rot_half + i + 1];
+        const float a = v.z, b = v.w;
+        v.z = fmaf(a, cs.x, -b * cs.y), v.w = fmaf(b, cs.x, a * cs.y);
+      }
+    }
+    put4<T>(q_full + (size_t)rh * hd + kv_rank + j, v.x, v.y, v.z, v.w);
+  }
+}
 }  // namespace
 
 LLM_EXPORT int llm_latent_store(float* proj, int proj_stride, const float* wq, const float* wc,
@@ -146,6 +193,20 @@ LLM_EXPORT int llm_latent_query(float* q, int q_stride, const float* cos_sin, in
   const long long total = (long long)rows * H * (dim + rot_dim);
   if (total <= 0) return 0;
   if (2 * rot_half > rot_dim) return LLM_ERR_ARGUMENT;
+  if ((dim & 3) == 0 && (rot_dim & 3) == 0 && (kv_rank & 3) == 0 && (q_stride & 3) == 0 && total < (1LL << 33) &&
+      (((uintptr_t)q | (uintptr_t)q_plain | (uintptr_t)q_full) & 15) == 0) {
+    const unsigned pieces = (unsigned)(total >> 2);
+    const int vblocks = (int)((pieces + 255) / 256 < 4736 ? (pieces + 255) / 256 : 4736);
+    if (dtype == LLM_F32)
+      return launched_many_blocks(
+          launch_pdl(latent_query_vec_kernel<float>, vblocks, 256, 0, stream, q, q_stride, (const float2*)cos_sin,
+                     rot_half, (float*)q_plain, (float*)q_full, pieces, H, dim, rot_dim, kv_rank, clear), vblocks);
+    if (dtype == LLM_BF16)
+      return launched_many_blocks(
+          launch_pdl(latent_query_vec_kernel<bf16>, vblocks, 256, 0, stream, q, q_stride, (const float2*)cos_sin,
+                     rot_half, (bf16*)q_plain, (bf16*)q_full, pieces, H, dim, rot_dim, kv_rank, clear), vblocks);
+    return LLM_ERR_UNSUPPORTED;
+  }
   const int blocks = (int)((total + 255) / 256 < 2368 ? (total + 255) / 256 : 2368);
   if (dtype == LLM_F32)
     return launched_many_blocks(

@@ -113,18 +113,29 @@ __global__ void __launch_bounds__(256) moe_router_kernel(const T* __restrict__ h
                                                          int top, int mode, const float* __restrict__ corr,
                                                          int* __restrict__ ids, float* __restrict__ wts,
                                                          float wscale) {
-  extern __shared__ float rs[];        // h[R][width], z[R][n_out]
+  extern __shared__ __align__(16) float rs[];        // h[R][width], z[R][n_out]
   float* h_s = rs;
   float* z_s = rs + (size_t)R * width;
   pdl_trigger();
   pdl_wait();
   const int r0 = blockIdx.x * R, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
+  const bool wide = (width & 3) == 0 && ((uintptr_t)w & 15) == 0;
+  if (sizeof(T) == 2 && (width & 7) == 0 && ((uintptr_t)h & 15) == 0) {
+    for (int i = threadIdx.x * 8; i < R * width; i += blockDim.x * 8) {     // (a piece stays inside its row)
+      const uint4 u = r0 + i / width < rows ? *reinterpret_cast<const uint4*>(h + (size_t)r0 * width + i)
+                                            : make_uint4(0, 0, 0, 0);
+      float4* dst = reinterpret_cast<float4*>(h_s + i);
+      dst[0] = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                           __uint_as_float(u.y & 0xffff0000u));
+      dst[1] = make_float4(__uint_as_float(u.z << 16), __uint_as_float(u.z & 0xffff0000u), __uint_as_float(u.w << 16),
+                           __uint_as_float(u.w & 0xffff0000u));
+    }
+  } else
   for (int i = threadIdx.x; i < R * width; i += blockDim.x) {
     const int rr = i / width, c = i - rr * width;
     h_s[i] = r0 + rr < rows ? to_f32(h[(size_t)(r0 + rr) * width + c]) : 0.f;
   }
   __syncthreads();
-  const bool wide = (width & 3) == 0 && ((uintptr_t)w & 15) == 0;
   for (int e = warp; e < n_out; e += nwarps) {
     const float* we = w + (size_t)e * width;
     float acc[R];
@@ -136,9 +147,9 @@ __global__ void __launch_bounds__(256) moe_router_kernel(const T* __restrict__ h
         const float4 a = *reinterpret_cast<const float4*>(we + i);
 #pragma unroll
         for (int rr = 0; rr < R; ++rr) {
-          const float* hr = h_s + (size_t)rr * width + i;
-          acc[rr] = fmaf(a.x, hr[0], acc[rr]), acc[rr] = fmaf(a.y, hr[1], acc[rr]);
-          acc[rr] = fmaf(a.z, hr[2], acc[rr]), acc[rr] = fmaf(a.w, hr[3], acc[rr]);
+          const float4 x = *reinterpret_cast<const float4*>(h_s + (size_t)rr * width + i);
+          acc[rr] = fmaf(a.x, x.x, acc[rr]), acc[rr] = fmaf(a.y, x.y, acc[rr]);
+          acc[rr] = fmaf(a.z, x.z, acc[rr]), acc[rr] = fmaf(a.w, x.w, acc[rr]);
         }
       }
     } else {

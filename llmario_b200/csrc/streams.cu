@@ -209,7 +209,9 @@ int launch_step(const StreamArgs& p, void* out, int rows, cudaStream_t stream) {
   const bool vec = (p.width & 3) == 0 && (p.stream_stride & 3) == 0 &&
                    (((uintptr_t)p.xs | (uintptr_t)p.y | (uintptr_t)p.w) & 15) == 0;
   if (vec) {
-    int threads = ((p.width >> 2) + 31) & ~31;
+    // few rows: a thread per four columns, so that a row is one round trip to memory; many rows: four
+    // times fewer, with four requests each under way and more rows on an SM
+    int threads = ((p.width >> (rows >= 512 ? 4 : 2)) + 31) & ~31;
     threads = threads < 128 ? 128 : (threads > 1024 ? 1024 : threads);
     if (p.y == nullptr || p.store || p.width <= 4 * KEEP4 * threads) {
 #define STEPV(N) \

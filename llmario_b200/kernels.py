@@ -1446,27 +1446,24 @@ def attention_latent_ok(dtype: torch.dtype, key_dim: int, value_dim: int, page_s
                                                                      page_size) > 0
 
 
-HEAD_LINEAR_SIMT_ROWS = 128     # up to so many rows the per-head maps are one CUDA-core launch
-
-
 def head_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
     """A map per head: ``out[r, h, :] = w[h] @ a[r, h, :]``.  a [rows, H, in] and out
     [rows, H, out_features] may be views with a row stride and a head stride (the last dimension dense); w
-    [H, out_features, in] contiguous.  Many rows of bfloat16 operands whose rows are whole
-    16-byte units go to the tensor-core product head by head; few rows (a launch per head would
-    cost more than the arithmetic) and everything else to one batched CUDA-core launch."""
+    [H, out_features, in] contiguous.  One launch either way: bfloat16 operands whose rows are whole
+    16-byte units on the tensor cores, everything else on the CUDA cores."""
     _cuda(a, w, out)
     rows, H, k = a.shape
     n = w.shape[1]
     assert w.shape == (H, n, k) and w.is_contiguous() and out.shape == (rows, H, n)
     assert a.stride(2) == 1 and out.stride(2) == 1 and a.dtype == w.dtype
-    if (rows > HEAD_LINEAR_SIMT_ROWS and a.dtype == torch.bfloat16 and k % 8 == 0
+    if (a.dtype == torch.bfloat16 and k % 8 == 0
             and a.stride(0) % 8 == 0 and a.stride(1) % 8 == 0 and a.data_ptr() % 16 == 0
             and w.data_ptr() % 16 == 0 and out.stride(1) >= n):
         # every head's product in one launch of the tensor-core kernel (its one-CTA form:
         # a head's product is small)
         _check(lib().llm_gemm_tcgen05_batched(_ptr(a), _ptr(w), _ptr(out), _dt(out), rows, n, k,
-                                              a.stride(0), k, out.stride(0), 128, H, a.stride(1),
+                                              a.stride(0), k, out.stride(0),
+                                              min(128, token_tile(rows)), H, a.stride(1),
                                               out.stride(1), _ptr(tc_status(a.device)),
                                               _stream()), "head_linear")
         return
