@@ -19,7 +19,7 @@ namespace {
 // channels behind the latent are never written and stay zero.  clear_proj: the row of proj that
 // was read is zeroed at the end (it lies in a buffer that a split-K product adds into).
 template <typename T>
-__global__ void __launch_bounds__(128) latent_store_kernel(
+__global__ void __launch_bounds__(512) latent_store_kernel(
     float* __restrict__ proj, int proj_stride, const float* __restrict__ wq, const float* __restrict__ wc,
     const float2* __restrict__ cos_sin, int rot_half, T* __restrict__ cq_out, T* __restrict__ k_plane,
     T* __restrict__ v_plane, long long page_stride, const int* __restrict__ block_table, int table_stride,
@@ -174,13 +174,16 @@ LLM_EXPORT int llm_latent_store(float* proj, int proj_stride, const float* wq, c
                                 cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (q_rank <= 0 || kv_rank <= 0 || rot_dim < 0 || 2 * rot_half > rot_dim) return LLM_ERR_ARGUMENT;
+  // few rows: a row is a chain of round trips to memory, shorter with more threads
+  const int most = rows < 512 ? 512 : 256, longest = q_rank > kv_rank ? q_rank : kv_rank;
+  const int threads = longest >= most ? most : longest > 128 ? (longest + 31) / 32 * 32 : 128;
   if (dtype == LLM_F32)
-    return launched_many_blocks(launch_pdl(latent_store_kernel<float>, rows, 128, 0, stream, proj, proj_stride, wq, wc,
+    return launched_many_blocks(launch_pdl(latent_store_kernel<float>, rows, threads, 0, stream, proj, proj_stride, wq, wc,
                       (const float2*)cos_sin, rot_half, (float*)cq_out, (float*)k_plane, (float*)v_plane,
                       page_stride, block_table, table_stride, row_slot, row_pos, page_size, q_rank, kv_rank,
                       rot_dim, eps, write_cache, clear_proj), rows);
   if (dtype == LLM_BF16)
-    return launched_many_blocks(launch_pdl(latent_store_kernel<bf16>, rows, 128, 0, stream, proj, proj_stride, wq, wc,
+    return launched_many_blocks(launch_pdl(latent_store_kernel<bf16>, rows, threads, 0, stream, proj, proj_stride, wq, wc,
                       (const float2*)cos_sin, rot_half, (bf16*)cq_out, (bf16*)k_plane, (bf16*)v_plane,
                       page_stride, block_table, table_stride, row_slot, row_pos, page_size, q_rank, kv_rank,
                       rot_dim, eps, write_cache, clear_proj), rows);

@@ -355,7 +355,8 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const float* __restric
   pdl_wait();
   const int r = blockIdx.x;
   const float g = shared ? 1.f / (1.f + expf(-gate[(size_t)r * gate_stride])) : 0.f;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+  // (a row's columns are shared by gridDim.y blocks when there are few rows)
+  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < width; c += blockDim.x * gridDim.y) {
     float sum = 0.f;
     for (int k = 0; k < top; ++k) {
       // (with ids: an expert behind the E with matrices is the identity, its output the row of x_id)
@@ -405,7 +406,8 @@ LLM_EXPORT int llm_moe_combine(const float* d, const int* pos, const float* wts,
                                int x_dtype, int x_stride, cudaStream_t stream) {
   if (rows <= 0) return 0;
   if ((shared && !gate) || (ids && !x_id)) return LLM_ERR_ARGUMENT;
-  return launched_many_blocks(launch_pdl(moe_combine_kernel, rows, 256, 0, stream, d, pos, wts, shared, gate,
+  const int per_row = rows < 256 && width <= 256 * 65535 ? (width + 255) / 256 : 1;
+  return launched_many_blocks(launch_pdl(moe_combine_kernel, dim3(rows, per_row), 256, 0, stream, d, pos, wts, shared, gate,
                                          gate_stride, y, width, top, accumulate, clear_shared, ids, E, x_id,
                                          x_dtype, x_stride), rows);
 }
