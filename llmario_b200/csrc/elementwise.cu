@@ -45,67 +45,78 @@ LLM_EXPORT int llm_embed(const int* tokens, const void* table, int table_dtype, 
   return llm_embed_scaled(tokens, table, table_dtype, x, rows, width, vocab, err_flag, 1.f, stream);
 }
 
-// y[r][:] = x[src(r)][:] * rsqrt(mean(x^2) + eps) * w[:]    sums and scale in 32-bit.
-// src(r) = rows_index ? rows_index[r] : r.
-template <typename TOut>
-__global__ void rms_norm_kernel(const float* __restrict__ x, const float* __restrict__ w,
-                                TOut* __restrict__ y, const int* __restrict__ rows_index, int width,
-                                float eps) {
+// RMS norm  y[r][:] = x[src(r)][:] * rsqrt(mean(x^2) + eps) * w[:]  and, with CENTRE, layer norm
+// y = (x - mean(x)) * rsqrt(mean((x - mean(x))^2) + eps) * w + b; sums and scale in 32-bit, the
+// deviations summed in a pass of their own behind the mean.  src(r) = rows_index ? rows_index[r] : r.
+template <typename TOut, bool CENTRE>
+__global__ void row_norm_kernel(const float* __restrict__ x, const float* __restrict__ w,
+                                const float* __restrict__ b, TOut* __restrict__ y,
+                                const int* __restrict__ rows_index, int width, float eps) {
   __shared__ float scratch[33];
   pdl_trigger();
   pdl_wait();
   const int r = blockIdx.x;
   const float* xr = x + (size_t)(rows_index ? rows_index[r] : r) * width;
+  float mean = 0.f;
+  if (CENTRE) {
+    for (int i = threadIdx.x; i < width; i += blockDim.x) mean += xr[i];
+    mean = block_sum(mean, scratch) / (float)width;
+  }
   float ss = 0.f;
   for (int i = threadIdx.x; i < width; i += blockDim.x) {
-    const float v = xr[i];
+    const float v = CENTRE ? xr[i] - mean : xr[i];
     ss += v * v;
   }
   ss = block_sum(ss, scratch);
   const float scale = 1.0f / sqrtf(ss / (float)width + eps);
-  for (int i = threadIdx.x; i < width; i += blockDim.x)
-    y[(size_t)r * width + i] = from_f32<TOut>(xr[i] * scale * w[i]);
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    const float v = CENTRE ? (xr[i] - mean) * scale * w[i] + b[i] : xr[i] * scale * w[i];
+    y[(size_t)r * width + i] = from_f32<TOut>(v);
+  }
 }
 
-// The same for widths that are multiples of four and at most 256 * 4 * VEC_MAX: the row is read
-// once with 16-byte loads and kept in registers between the sum and the scaling.
-constexpr int VEC_MAX = 8;
-template <typename TOut>
-__global__ void __launch_bounds__(256) rms_norm_vec_kernel(const float* __restrict__ x,
-                                                           const float* __restrict__ w, TOut* __restrict__ y,
-                                                           const int* __restrict__ rows_index, int width,
-                                                           float eps) {
-  __shared__ float scratch[33];
-  pdl_trigger();
-  pdl_wait();
-  const int r = blockIdx.x;
-  const float4* xr = reinterpret_cast<const float4*>(x + (size_t)(rows_index ? rows_index[r] : r) * width);
-  const float4* wr = reinterpret_cast<const float4*>(w);
-  const int n4 = width >> 2;
-  float4 v[VEC_MAX];
+// The same for widths that are multiples of four, of a row that its threads keep in registers
+// between the sums and the scaling: thread `at` of `stride` holds the float4 pieces at, at + stride, ...
+template <int N, bool CENTRE, typename Sum>
+__device__ __forceinline__ float row_norm_scale(float4 (&v)[N], const float4* __restrict__ xr, int at, int stride,
+                                                int n4, int width, float eps, Sum sum) {
+#pragma unroll
+  for (int k = 0; k < N; ++k)
+    if (at + k * stride < n4) v[k] = xr[at + k * stride];
+  if (CENTRE) {
+    float mean = 0.f;
+#pragma unroll
+    for (int k = 0; k < N; ++k)
+      if (at + k * stride < n4) mean += (v[k].x + v[k].y) + (v[k].z + v[k].w);
+    mean = sum(mean) / (float)width;
+#pragma unroll
+    for (int k = 0; k < N; ++k) v[k].x -= mean, v[k].y -= mean, v[k].z -= mean, v[k].w -= mean;
+  }
   float ss = 0.f;
 #pragma unroll
-  for (int k = 0; k < VEC_MAX; ++k) {
-    const int i = threadIdx.x + k * 256;
-    if (i < n4) {
-      v[k] = xr[i];
-      ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
-    }
-  }
-  ss = block_sum(ss, scratch);
-  const float scale = 1.0f / sqrtf(ss / (float)width + eps);
+  for (int k = 0; k < N; ++k)
+    if (at + k * stride < n4) ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+  return 1.0f / sqrtf(sum(ss) / (float)width + eps);
+}
+template <typename TOut, int N, bool CENTRE>
+__device__ __forceinline__ void row_norm_write(const float4 (&v)[N], float scale, const float* __restrict__ w,
+                                               const float* __restrict__ b, TOut* __restrict__ yr, int at, int stride,
+                                               int n4) {
 #pragma unroll
-  for (int k = 0; k < VEC_MAX; ++k) {
-    const int i = threadIdx.x + k * 256;
+  for (int k = 0; k < N; ++k) {
+    const int i = at + k * stride;
     if (i < n4) {
-      const float4 g = wr[i];
-      const float a = v[k].x * scale * g.x, b = v[k].y * scale * g.y, c = v[k].z * scale * g.z,
-                  d = v[k].w * scale * g.w;
-      TOut* dst = y + (size_t)r * width + 4 * i;
+      const float4 g = reinterpret_cast<const float4*>(w)[i];
+      float4 o = make_float4(v[k].x * scale * g.x, v[k].y * scale * g.y, v[k].z * scale * g.z, v[k].w * scale * g.w);
+      if (CENTRE) {
+        const float4 c = reinterpret_cast<const float4*>(b)[i];
+        o.x += c.x, o.y += c.y, o.z += c.z, o.w += c.w;
+      }
+      TOut* dst = yr + 4 * i;
       if (sizeof(TOut) == 4) {
-        *reinterpret_cast<float4*>(dst) = make_float4(a, b, c, d);
+        *reinterpret_cast<float4*>(dst) = o;
       } else {
-        __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
+        __nv_bfloat162 lo = __floats2bfloat162_rn(o.x, o.y), hi = __floats2bfloat162_rn(o.z, o.w);
         uint2 packed;
         packed.x = *reinterpret_cast<uint32_t*>(&lo);
         packed.y = *reinterpret_cast<uint32_t*>(&hi);
@@ -113,6 +124,23 @@ __global__ void __launch_bounds__(256) rms_norm_vec_kernel(const float* __restri
       }
     }
   }
+}
+
+// A block per row of at most 256 * 4 * VEC_MAX values.
+constexpr int VEC_MAX = 8;
+template <typename TOut, bool CENTRE>
+__global__ void __launch_bounds__(256) row_norm_vec_kernel(const float* __restrict__ x, const float* __restrict__ w,
+                                                           const float* __restrict__ b, TOut* __restrict__ y,
+                                                           const int* __restrict__ rows_index, int width, float eps) {
+  __shared__ float scratch[33];
+  pdl_trigger();
+  pdl_wait();
+  const int r = blockIdx.x, n4 = width >> 2;
+  const float4* xr = reinterpret_cast<const float4*>(x + (size_t)(rows_index ? rows_index[r] : r) * width);
+  float4 v[VEC_MAX];
+  const float scale = row_norm_scale<VEC_MAX, CENTRE>(v, xr, threadIdx.x, 256, n4, width, eps,
+                                                      [&](float s) { return block_sum(s, scratch); });
+  row_norm_write<TOut, VEC_MAX, CENTRE>(v, scale, w, b, y + (size_t)r * width, threadIdx.x, 256, n4);
 }
 
 // Many rows of a narrow width (at most 32 * 4 * WARP_VEC values): a warp per row, eight rows per
@@ -120,79 +148,55 @@ __global__ void __launch_bounds__(256) rms_norm_vec_kernel(const float* __restri
 // per thread and two barriers, and the kernel is bound by launching blocks (8.6 us for 2,048
 // rows of 1,024 against 3 us here).
 constexpr int WARP_VEC = 16;
-template <typename TOut>
-__global__ void __launch_bounds__(256) rms_norm_warp_kernel(const float* __restrict__ x,
-                                                            const float* __restrict__ w, TOut* __restrict__ y,
-                                                            const int* __restrict__ rows_index, int rows,
-                                                            int width, float eps) {
+template <typename TOut, bool CENTRE>
+__global__ void __launch_bounds__(256) row_norm_warp_kernel(const float* __restrict__ x, const float* __restrict__ w,
+                                                            const float* __restrict__ b, TOut* __restrict__ y,
+                                                            const int* __restrict__ rows_index, int rows, int width,
+                                                            float eps) {
   pdl_trigger();
   pdl_wait();
-  const int r = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int r = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, n4 = width >> 2;
   if (r >= rows) return;
   const float4* xr = reinterpret_cast<const float4*>(x + (size_t)(rows_index ? rows_index[r] : r) * width);
-  const float4* wr = reinterpret_cast<const float4*>(w);
-  const int n4 = width >> 2;
   float4 v[WARP_VEC];
-  float ss = 0.f;
-#pragma unroll
-  for (int k = 0; k < WARP_VEC; ++k) {
-    const int i = lane + k * 32;
-    if (i < n4) {
-      v[k] = xr[i];
-      ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
-    }
-  }
-  ss = warp_sum(ss);
-  const float scale = 1.0f / sqrtf(ss / (float)width + eps);
-#pragma unroll
-  for (int k = 0; k < WARP_VEC; ++k) {
-    const int i = lane + k * 32;
-    if (i < n4) {
-      const float4 g = wr[i];
-      const float a = v[k].x * scale * g.x, b = v[k].y * scale * g.y, c = v[k].z * scale * g.z,
-                  d = v[k].w * scale * g.w;
-      TOut* dst = y + (size_t)r * width + 4 * i;
-      if (sizeof(TOut) == 4) {
-        *reinterpret_cast<float4*>(dst) = make_float4(a, b, c, d);
-      } else {
-        __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
-        uint2 packed;
-        packed.x = *reinterpret_cast<uint32_t*>(&lo);
-        packed.y = *reinterpret_cast<uint32_t*>(&hi);
-        *reinterpret_cast<uint2*>(dst) = packed;
-      }
-    }
-  }
+  const float scale = row_norm_scale<WARP_VEC, CENTRE>(v, xr, lane, 32, n4, width, eps,
+                                                       [](float s) { return warp_sum(s); });
+  row_norm_write<TOut, WARP_VEC, CENTRE>(v, scale, w, b, y + (size_t)r * width, lane, 32, n4);
+}
+
+template <typename TOut, bool CENTRE>
+static int launch_row_norm(const float* x, const float* w, const float* b, TOut* y, const int* rows_index, int rows,
+                           int width, float eps, cudaStream_t stream) {
+  const bool vec = width % 4 == 0 && width <= 256 * 4 * VEC_MAX &&
+                   (((uintptr_t)x | (uintptr_t)w | (uintptr_t)b | (uintptr_t)y) & 15) == 0;
+  if (vec && rows >= 512 && width <= 32 * 4 * WARP_VEC)
+    return launch_pdl(row_norm_warp_kernel<TOut, CENTRE>, (rows + 7) / 8, 256, 0, stream, x, w, b, y, rows_index,
+                      rows, width, eps);
+  if (vec)
+    return launch_pdl(row_norm_vec_kernel<TOut, CENTRE>, rows, 256, 0, stream, x, w, b, y, rows_index, width, eps);
+  const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
+  return launch_pdl(row_norm_kernel<TOut, CENTRE>, rows, threads, 0, stream, x, w, b, y, rows_index, width, eps);
 }
 
 LLM_EXPORT int llm_rms_norm(const float* x, const float* w, void* y, int out_dtype,
                             const int* rows_index, int rows, int width, float eps,
                             cudaStream_t stream) {
   if (rows <= 0) return 0;
-  const bool vec = width % 4 == 0 && width <= 256 * 4 * VEC_MAX &&
-                   (((uintptr_t)x | (uintptr_t)w | (uintptr_t)y) & 15) == 0;
-  if (vec && rows >= 512 && width <= 32 * 4 * WARP_VEC) {
-    const int blocks = (rows + 7) / 8;
-    if (out_dtype == LLM_F32)
-      return launch_pdl(rms_norm_warp_kernel<float>, blocks, 256, 0, stream, x, w, (float*)y, rows_index, rows,
-                        width, eps);
-    if (out_dtype == LLM_BF16)
-      return launch_pdl(rms_norm_warp_kernel<bf16>, blocks, 256, 0, stream, x, w, (bf16*)y, rows_index, rows,
-                        width, eps);
-    return LLM_ERR_UNSUPPORTED;
-  }
-  if (vec) {
-    if (out_dtype == LLM_F32)
-      return launch_pdl(rms_norm_vec_kernel<float>, rows, 256, 0, stream, x, w, (float*)y, rows_index, width, eps);
-    if (out_dtype == LLM_BF16)
-      return launch_pdl(rms_norm_vec_kernel<bf16>, rows, 256, 0, stream, x, w, (bf16*)y, rows_index, width, eps);
-    return LLM_ERR_UNSUPPORTED;
-  }
-  const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
   if (out_dtype == LLM_F32)
-    return launch_pdl(rms_norm_kernel<float>, rows, threads, 0, stream, x, w, (float*)y, rows_index, width, eps);
+    return launch_row_norm<float, false>(x, w, nullptr, (float*)y, rows_index, rows, width, eps, stream);
   if (out_dtype == LLM_BF16)
-    return launch_pdl(rms_norm_kernel<bf16>, rows, threads, 0, stream, x, w, (bf16*)y, rows_index, width, eps);
+    return launch_row_norm<bf16, false>(x, w, nullptr, (bf16*)y, rows_index, rows, width, eps, stream);
+  return LLM_ERR_UNSUPPORTED;
+}
+
+LLM_EXPORT int llm_layer_norm(const float* x, const float* w, const float* b, void* y, int out_dtype,
+                              const int* rows_index, int rows, int width, float eps, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (width <= 0 || w == nullptr || b == nullptr) return LLM_ERR_ARGUMENT;
+  if (out_dtype == LLM_F32)
+    return launch_row_norm<float, true>(x, w, b, (float*)y, rows_index, rows, width, eps, stream);
+  if (out_dtype == LLM_BF16)
+    return launch_row_norm<bf16, true>(x, w, b, (bf16*)y, rows_index, rows, width, eps, stream);
   return LLM_ERR_UNSUPPORTED;
 }
 

@@ -19,6 +19,10 @@
 
 namespace {
 constexpr int MAX_TOP = 16;
+constexpr int MAX_GROUPS = 1024;
+
+// Experts in groups of `size` neighbours of which only the `keep` best can be chosen; keep 0: no groups.
+struct Groups { int size, keep; };
 
 // The choice of one row by one warp, from its E router outputs zr (shared or global memory).
 // mode 0: the k-th choice is the largest logit not chosen before (the lowest index among equals);
@@ -27,9 +31,12 @@ constexpr int MAX_TOP = 16;
 // of a chosen expert is its score, not renormalised.  mode 2: as mode 1, but the weights are the
 // chosen scores over their sum (+ 1e-20), times `wscale`.  mode 3: the choice as in mode 0 (the sigmoid
 // keeps the order of the logits); the weight of a chosen expert is the sigmoid of its own logit.
+// With groups only experts of the `keep` best groups take part in the choice, a group's worth being
+// the largest of what its experts are chosen by (the lowest index among equals); scores that go
+// over all outputs still do.
 __device__ __forceinline__ void choose_row(const float* zr, int E, int top, int mode, const float* __restrict__ corr,
                                            int lane, int* __restrict__ ids, float* __restrict__ wts,
-                                           float wscale = 1.f) {
+                                           float wscale, Groups groups) {
   const bool renorm = mode == 2;
   if (renorm) mode = 1;
   float zmax = 0.f, inv_sum = 1.f;
@@ -41,23 +48,52 @@ __device__ __forceinline__ void choose_row(const float* zr, int E, int top, int 
     for (int e = lane; e < E; e += 32) sum += expf(zr[e] - zmax);
     inv_sum = 1.f / warp_sum(sum);
   }
-  float best[MAX_TOP];
-  int pick[MAX_TOP];
-  for (int k = 0; k < top; ++k) {
-    float v = -INFINITY;
-    int at = 0x7fffffff;
-    for (int e = lane; e < E; e += 32) {
-      bool taken = false;
-      for (int j = 0; j < k; ++j) taken |= pick[j] == e;
-      const float x = mode == 1 ? expf(zr[e] - zmax) * inv_sum + (corr ? corr[e] : 0.f) : zr[e];
-      if (!taken && (x > v || (x == v && e < at) || at == 0x7fffffff)) v = x, at = e;
-    }
+  constexpr int NONE = 0x7fffffff;
+  auto worth = [&](int e) { return mode == 1 ? expf(zr[e] - zmax) * inv_sum + (corr ? corr[e] : 0.f) : zr[e]; };
+  auto take = [&](float x, int e, float& v, int& at) {      // (v, at) <- the better of it and (x, e)
+    if (e != NONE && (at == NONE || x > v || (x == v && e < at))) v = x, at = e;
+  };
+  auto best_of_warp = [&](float& v, int& at) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       const float ov = __shfl_xor_sync(0xffffffffu, v, o);
       const int oa = __shfl_xor_sync(0xffffffffu, at, o);
-      if (oa != 0x7fffffff && (at == 0x7fffffff || ov > v || (ov == v && oa < at))) v = ov, at = oa;
+      take(ov, oa, v, at);
     }
+  };
+  unsigned open = 0xffffffffu;       // bit j of lane l: experts of group l + 32 j can be chosen
+  if (groups.keep > 0) {
+    open = 0;
+    const int count = E / groups.size;
+    for (int k = 0; k < groups.keep; ++k) {
+      float v = -INFINITY;
+      int at = NONE;
+      for (int g = lane; g < count; g += 32) {
+        if ((open >> (g >> 5)) & 1u) continue;
+        float m = worth(g * groups.size);
+        for (int j = 1; j < groups.size; ++j) m = fmaxf(m, worth(g * groups.size + j));
+        take(m, g, v, at);
+      }
+      best_of_warp(v, at);
+      if (at != NONE && (at & 31) == lane) open |= 1u << (at >> 5);
+    }
+  }
+  float best[MAX_TOP];
+  int pick[MAX_TOP];
+  for (int k = 0; k < top; ++k) {
+    float v = -INFINITY;
+    int at = NONE;
+    for (int e0 = 0; e0 < E; e0 += 32) {       // (all lanes together: they hold the groups' bits)
+      const int e = e0 + lane;
+      bool free = e < E;
+      if (groups.keep > 0) {
+        const int g = (free ? e : E - 1) / groups.size;
+        free = ((__shfl_sync(0xffffffffu, open, g & 31) >> (g >> 5)) & 1u) && free;
+      }
+      for (int j = 0; j < k; ++j) free = free && pick[j] != e;
+      if (free) take(worth(e), e, v, at);
+    }
+    best_of_warp(v, at);
     best[k] = v, pick[k] = at;
   }
   if (lane == 0) {
@@ -91,13 +127,13 @@ __device__ __forceinline__ void choose_row(const float* zr, int E, int top, int 
 __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ z, int z_stride, int rows, int E,
                                                         int top, int mode, const float* __restrict__ corr,
                                                         int* __restrict__ ids, float* __restrict__ wts,
-                                                        float wscale) {
+                                                        float wscale, Groups groups) {
   pdl_trigger();
   pdl_wait();
   const int r = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (r >= rows) return;
   choose_row(z + (size_t)r * z_stride, E, top, mode, corr, lane, ids + (size_t)r * top, wts + (size_t)r * top,
-             wscale);
+             wscale, groups);
 }
 
 
@@ -112,7 +148,7 @@ __global__ void __launch_bounds__(256) moe_router_kernel(const T* __restrict__ h
                                                          int z_stride, int rows, int width, int E, int n_out,
                                                          int top, int mode, const float* __restrict__ corr,
                                                          int* __restrict__ ids, float* __restrict__ wts,
-                                                         float wscale) {
+                                                         float wscale, Groups groups) {
   extern __shared__ __align__(16) float rs[];        // h[R][width], z[R][n_out]
   float* h_s = rs;
   float* z_s = rs + (size_t)R * width;
@@ -172,7 +208,8 @@ __global__ void __launch_bounds__(256) moe_router_kernel(const T* __restrict__ h
   __syncthreads();
   if (warp >= R || r0 + warp >= rows) return;
   const int r = r0 + warp;
-  choose_row(z_s + warp * n_out, E, top, mode, corr, lane, ids + (size_t)r * top, wts + (size_t)r * top, wscale);
+  choose_row(z_s + warp * n_out, E, top, mode, corr, lane, ids + (size_t)r * top, wts + (size_t)r * top, wscale,
+             groups);
 }
 
 template <typename T> __device__ __forceinline__ float dot_row(const T* __restrict__ w, const float* __restrict__ x,
@@ -412,15 +449,24 @@ LLM_EXPORT int llm_moe_combine(const float* d, const int* pos, const float* wts,
                                          x_dtype, x_stride), rows);
 }
 
+// Whether `keep` of the groups of `size` neighbours of E experts hold `top` of them (keep 0: no groups).
+static bool groups_ok(int E, int top, int size, int keep) {
+  if (keep == 0) return true;
+  return size > 0 && keep > 0 && E % size == 0 && E / size <= MAX_GROUPS && keep <= E / size &&
+         (long long)keep * size >= top;
+}
+
 // The router: z_out[r][0:n_out] = w h_r + b (w float32 [n_out][width], the first E rows the
 // experts'), ids / wts the `top` chosen experts of every row and their weights.
-// mode and corr: see choose_row.
-// mode, corr and wscale: see choose_row.
-LLM_EXPORT int llm_moe_router_scaled(const void* h, int dtype, const float* w, const float* b, float* z_out,
+// mode, corr, wscale and the groups (group_size, keep; keep 0: none): see choose_row.
+LLM_EXPORT int llm_moe_router_groups(const void* h, int dtype, const float* w, const float* b, float* z_out,
                                      int z_stride, int rows, int width, int E, int n_out, int top, int mode,
-                                     const float* corr, int* ids, float* wts, float wscale, cudaStream_t stream) {
+                                     const float* corr, int* ids, float* wts, float wscale, int group_size, int keep,
+                                     cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (top < 1 || top > MAX_TOP || top > E || n_out < E || mode < 0 || mode > 3) return LLM_ERR_UNSUPPORTED;
+  if (!groups_ok(E, top, group_size, keep)) return LLM_ERR_ARGUMENT;
+  const Groups groups = {group_size, keep};
   if ((size_t)(width + n_out) * 4 > 200 * 1024) return LLM_ERR_UNSUPPORTED;
   // many rows: four to a block, so that a block reads the router's rows once for four tokens
   const bool four = rows >= 256 && (size_t)4 * (width + n_out) * 4 <= 200 * 1024;
@@ -432,7 +478,7 @@ LLM_EXPORT int llm_moe_router_scaled(const void* h, int dtype, const float* w, c
     if (smem > 48 * 1024)                                                                                      \
       cudaFuncSetAttribute(moe_router_kernel<T, RR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);  \
     return launch_pdl(moe_router_kernel<T, RR>, blocks, 256, smem, stream, (const T*)h, w, b, z_out, z_stride, \
-                      rows, width, E, n_out, top, mode, corr, ids, wts, wscale);                               \
+                      rows, width, E, n_out, top, mode, corr, ids, wts, wscale, groups);                       \
   } while (0)
   if (dtype == LLM_F32) {
     if (four) ROUTER(float, 4);
@@ -446,6 +492,13 @@ LLM_EXPORT int llm_moe_router_scaled(const void* h, int dtype, const float* w, c
   return LLM_ERR_UNSUPPORTED;
 }
 
+LLM_EXPORT int llm_moe_router_scaled(const void* h, int dtype, const float* w, const float* b, float* z_out,
+                                     int z_stride, int rows, int width, int E, int n_out, int top, int mode,
+                                     const float* corr, int* ids, float* wts, float wscale, cudaStream_t stream) {
+  return llm_moe_router_groups(h, dtype, w, b, z_out, z_stride, rows, width, E, n_out, top, mode, corr, ids, wts,
+                               wscale, 0, 0, stream);
+}
+
 LLM_EXPORT int llm_moe_router(const void* h, int dtype, const float* w, const float* b, float* z_out, int z_stride,
                               int rows, int width, int E, int n_out, int top, int mode, const float* corr,
                               int* ids, float* wts, cudaStream_t stream) {
@@ -453,12 +506,20 @@ LLM_EXPORT int llm_moe_router(const void* h, int dtype, const float* w, const fl
                                1.f, stream);
 }
 
-LLM_EXPORT int llm_moe_route_scaled(const float* z, int z_stride, int rows, int E, int top, int mode,
-                                    const float* corr, int* ids, float* wts, float wscale, cudaStream_t stream) {
+LLM_EXPORT int llm_moe_route_groups(const float* z, int z_stride, int rows, int E, int top, int mode,
+                                    const float* corr, int* ids, float* wts, float wscale, int group_size, int keep,
+                                    cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (top < 1 || top > MAX_TOP || top > E || mode < 0 || mode > 3) return LLM_ERR_UNSUPPORTED;
+  if (!groups_ok(E, top, group_size, keep)) return LLM_ERR_ARGUMENT;
+  const Groups groups = {group_size, keep};
   return launch_pdl(moe_route_kernel, (rows + 3) / 4, 128, 0, stream, z, z_stride, rows, E, top, mode, corr, ids,
-                    wts, wscale);
+                    wts, wscale, groups);
+}
+
+LLM_EXPORT int llm_moe_route_scaled(const float* z, int z_stride, int rows, int E, int top, int mode,
+                                    const float* corr, int* ids, float* wts, float wscale, cudaStream_t stream) {
+  return llm_moe_route_groups(z, z_stride, rows, E, top, mode, corr, ids, wts, wscale, 0, 0, stream);
 }
 
 LLM_EXPORT int llm_moe_route(const float* z, int z_stride, int rows, int E, int top, int mode, const float* corr,

@@ -13,6 +13,12 @@
 //   temperature: the queries of position p are multiplied by 1 + coef * ln(floor((p + 1) / every) + 1).
 //   blend: the value that is stored is (1 - lambda) v + lambda v0, v0 another layer's values of
 //   the same rows (32-bit, as projected).
+//   bias: added to q, k and v as they are read (not with norm 2).
+//   maps: a head has so many queries and keys of d channels over the same values (its q and k are
+//   laid out [map 0, map 1, ..]; norm and rotation per map).  The maps' keys of a head stand side by
+//   side in one cache row; map m's query is a row of its own, [rows][Hq * maps][hd], that holds its
+//   channels at m * d and zeros elsewhere: a dot product with the cache row is the map's score.
+//   clear: what was read is zeroed (a split-K product adds into it the next time; not with norm 2).
 //
 // llm_pool_blocks, one block per (row, key head): a row whose position ends a block of P tokens
 // (pos % P == P - 1) writes entry pos / P of the pooled cache: the means of the block's P cached
@@ -36,6 +42,8 @@ struct StoreArgs {
   float temp_coef; int temp_every;     // query temperature by position (every 0: none)
   const float* v0; int v0_stride;      // values to blend in ([rows][Hkv * dv]) or null
   float blend;
+  const float *q_b, *k_b, *v_b;        // biases or null
+  int maps, clear;
 };
 
 __device__ __forceinline__ void store2(float* dst, float a, float b) { *reinterpret_cast<float2*>(dst) = make_float2(a, b); }
@@ -82,49 +90,67 @@ __global__ void __launch_bounds__(256) qkv_store_kernel(const StoreArgs a) {
     page_off = (long long)page * a.page_stride;
   }
   const float* cs = a.cos_sin ? a.cos_sin + (size_t)r * (a.rot / 2) * 2 : nullptr;
-  const int heads = a.Hq + (a.has_kv ? 2 * a.Hkv : 0);
+  const int nq = a.Hq * a.maps, nk = a.Hkv * a.maps;      // query and key rows of d channels
+  const int heads = nq + (a.has_kv ? nk + a.Hkv : 0);
   for (int item = blockIdx.y * nwarps + warp; item < heads; item += nwarps * gridDim.y) {
-    if (item >= a.Hq + a.Hkv) {                    // a value head: a copy, padded with zeros
-      const int g = item - a.Hq - a.Hkv;
+    if (item >= nq + nk) {                         // a value head: a copy, padded with zeros
+      const int g = item - nq - nk;
       const float* src = a.v + (size_t)r * a.v_stride + (size_t)g * a.dv;
+      const float* bias = a.v_b ? a.v_b + (size_t)g * a.dv : nullptr;
       const float* mix = a.v0 ? a.v0 + (size_t)r * a.v0_stride + (size_t)g * a.dv : nullptr;
       const float keep = 1.f - a.blend;
       T* dst = (T*)a.v_cache + page_off + ((long long)g * a.page_size + pos % a.page_size) * a.hd;
       if (PAIRS && !mix) {
         for (int c = 2 * lane; c < a.hd; c += 64) {
           float2 x = make_float2(0.f, 0.f);
-          if (c < a.dv) x = *reinterpret_cast<const float2*>(src + c);
+          if (c < a.dv) {
+            x = *reinterpret_cast<const float2*>(src + c);
+            if (bias) x.x += bias[c], x.y += bias[c + 1];
+            if (a.clear) *reinterpret_cast<float2*>(const_cast<float*>(src) + c) = make_float2(0.f, 0.f);
+          }
           store2(dst + c, x.x, x.y);
         }
       } else {
         for (int c = lane; c < a.hd; c += 32) {
-          float x = c < a.dv ? src[c] : 0.f;
+          float x = c < a.dv ? src[c] + (bias ? bias[c] : 0.f) : 0.f;
+          if (a.clear && c < a.dv) const_cast<float*>(src)[c] = 0.f;
           if (mix && c < a.dv) x = fmaf(a.blend, mix[c], keep * x);
           dst[c] = from_f32<T>(x);
         }
       }
       continue;
     }
-    const bool is_q = item < a.Hq;
-    const int h = is_q ? item : item - a.Hq;
+    const bool is_q = item < nq;
+    const int h = is_q ? item : item - nq, m = h % a.maps;
     const float* src = (is_q ? qr : kr) + (size_t)h * a.d;
     const float* w = is_q ? a.q_w : a.k_w;
+    const float* bias = is_q ? a.q_b : a.k_b;
+    if (bias) bias += (size_t)h * a.d;
     float scale = is_q ? whole_q : whole_k;
     if (a.norm == 1) {
       float s = 0.f;
-      for (int c = lane; c < a.d; c += 32) s = fmaf(src[c], src[c], s);
-      scale = rsqrtf(warp_sum(s) / (float)a.d + a.eps);
+      for (int c = lane; c < a.d; c += 32) {
+        const float x = src[c] + (bias ? bias[c] : 0.f);
+        s = fmaf(x, x, s);
+      }
+      scale = 1.f / sqrtf(warp_sum(s) / (float)a.d + a.eps);
     }
     if (is_q) scale *= temp;
     if (w && a.norm == 2) w += (size_t)h * a.d;
     if (!a.norm) w = nullptr;
-    T* dst = is_q ? (T*)a.q_out + ((size_t)r * a.Hq + h) * a.hd
-                  : (T*)a.k_cache + page_off + ((long long)h * a.page_size + pos % a.page_size) * a.hd;
+    // the map's channels start at m * d of its row; a query fills its row, a key what is its own (the
+    // last map's also what is behind it)
+    T* dst = (is_q ? (T*)a.q_out + ((size_t)r * nq + h) * a.hd
+                   : (T*)a.k_cache + page_off + ((long long)(h / a.maps) * a.page_size + pos % a.page_size) * a.hd) +
+             m * a.d;
+    const int c0 = is_q ? -m * a.d : 0, c1 = is_q || m == a.maps - 1 ? a.hd - m * a.d : a.d;
     if (PAIRS) {
-      for (int c = 2 * lane; c < a.hd; c += 64) {
+      for (int c = c0 + 2 * lane; c < c1; c += 64) {
         float x = 0.f, y = 0.f;
-        if (c < a.d) {
-          const float2 u = *reinterpret_cast<const float2*>(src + c);
+        if (c >= 0 && c < a.d) {
+          float2 u = *reinterpret_cast<const float2*>(src + c);
+          if (bias) u.x += bias[c], u.y += bias[c + 1];
+          if (a.clear) *reinterpret_cast<float2*>(const_cast<float*>(src) + c) = make_float2(0.f, 0.f);
           x = u.x * scale * (w ? w[c] : 1.f);
           y = u.y * scale * (w ? w[c + 1] : 1.f);
           if (cs && c < a.rot) {
@@ -138,18 +164,22 @@ __global__ void __launch_bounds__(256) qkv_store_kernel(const StoreArgs a) {
       }
       continue;
     }
-    for (int c = lane; c < a.hd; c += 32) {
+    for (int c = c0 + lane; c < c1; c += 32) {
       float x = 0.f;
-      if (c < a.d) {
-        x = src[c] * scale * (w ? w[c] : 1.f);
+      if (c >= 0 && c < a.d) {
+        x = (src[c] + (bias ? bias[c] : 0.f)) * scale * (w ? w[c] : 1.f);
         if (cs && c < a.rot) {
           const int o = c ^ 1;                       // the other member of the pair
-          const float y = src[o] * scale * (w ? w[o] : 1.f);
+          const float y = (src[o] + (bias ? bias[o] : 0.f)) * scale * (w ? w[o] : 1.f);
           const float co = cs[(c >> 1) * 2], si = cs[(c >> 1) * 2 + 1];
           x = (c & 1) ? fmaf(x, co, y * si) : fmaf(x, co, -(y * si));
         }
       }
       dst[c] = from_f32<T>(x);
+    }
+    if (a.clear) {
+      __syncwarp();
+      for (int c = lane; c < a.d; c += 32) const_cast<float*>(src)[c] = 0.f;
     }
   }
 }
@@ -199,17 +229,20 @@ __global__ void __launch_bounds__(1024) pool_blocks_kernel(
 }
 }  // namespace
 
-LLM_EXPORT int llm_qkv_store_mix(const float* q, int q_stride, const float* k, int k_stride, const float* v,
-                                 int v_stride, const float* q_w, const float* k_w, const float* cos_sin,
-                                 void* q_out, void* k_cache, void* v_cache, int dtype, long long page_stride,
-                                 const int* table, int table_stride, const int* row_slot, const int* row_pos,
-                                 int rows, int Hq, int Hkv, int d, int dv, int hd, int rot, int norm, float eps,
-                                 int page_size, int has_kv, float temp_coef, int temp_every, const float* v0,
-                                 int v0_stride, float blend, cudaStream_t stream) {
+LLM_EXPORT int llm_qkv_store_maps(const float* q, int q_stride, const float* k, int k_stride, const float* v,
+                                  int v_stride, const float* q_w, const float* k_w, const float* cos_sin,
+                                  void* q_out, void* k_cache, void* v_cache, int dtype, long long page_stride,
+                                  const int* table, int table_stride, const int* row_slot, const int* row_pos,
+                                  int rows, int Hq, int Hkv, int d, int dv, int hd, int rot, int norm, float eps,
+                                  int page_size, int has_kv, float temp_coef, int temp_every, const float* v0,
+                                  int v0_stride, float blend, const float* q_b, const float* k_b, const float* v_b,
+                                  int maps, int clear, cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (temp_every < 0) return LLM_ERR_ARGUMENT;
-  if (d <= 0 || dv <= 0 || hd < d || hd < dv || rot < 0 || rot > d || (rot & 1) || norm < 0 || norm > 2)
+  if (d <= 0 || dv <= 0 || maps <= 0 || hd < maps * d || hd < dv || rot < 0 || rot > d || (rot & 1) || norm < 0 ||
+      norm > 2)
     return LLM_ERR_ARGUMENT;
+  if (norm == 2 && (q_b || k_b || v_b || maps > 1 || clear)) return LLM_ERR_ARGUMENT;
   if (rot > 0 && !cos_sin) return LLM_ERR_ARGUMENT;
   StoreArgs a;
   a.q = q, a.k = k, a.v = v, a.q_stride = q_stride, a.k_stride = k_stride, a.v_stride = v_stride;
@@ -220,7 +253,8 @@ LLM_EXPORT int llm_qkv_store_mix(const float* q, int q_stride, const float* k, i
   a.dv = dv, a.hd = hd, a.rot = rot, a.norm = norm, a.has_kv = has_kv, a.eps = eps;
   a.temp_coef = temp_coef, a.temp_every = temp_every, a.v0 = has_kv ? v0 : nullptr, a.v0_stride = v0_stride,
   a.blend = blend;
-  const int heads = Hq + (has_kv ? 2 * Hkv : 0);
+  a.q_b = q_b, a.k_b = k_b, a.v_b = v_b, a.maps = maps, a.clear = clear;
+  const int heads = Hq * maps + (has_kv ? (maps + 1) * Hkv : 0);
   const int threads = heads >= 8 ? 256 : heads >= 4 ? 128 : 64;
   // few rows: the heads of a row are shared out to several blocks, so that the step fills the GPU
   int shares = 1;
@@ -242,6 +276,19 @@ LLM_EXPORT int llm_qkv_store_mix(const float* q, int q_stride, const float* k, i
   else return LLM_ERR_UNSUPPORTED;
 #undef STORE_GO
   return launched_many_blocks(rc, (long long)rows * shares);
+}
+
+LLM_EXPORT int llm_qkv_store_mix(const float* q, int q_stride, const float* k, int k_stride, const float* v,
+                                 int v_stride, const float* q_w, const float* k_w, const float* cos_sin,
+                                 void* q_out, void* k_cache, void* v_cache, int dtype, long long page_stride,
+                                 const int* table, int table_stride, const int* row_slot, const int* row_pos,
+                                 int rows, int Hq, int Hkv, int d, int dv, int hd, int rot, int norm, float eps,
+                                 int page_size, int has_kv, float temp_coef, int temp_every, const float* v0,
+                                 int v0_stride, float blend, cudaStream_t stream) {
+  return llm_qkv_store_maps(q, q_stride, k, k_stride, v, v_stride, q_w, k_w, cos_sin, q_out, k_cache, v_cache, dtype,
+                            page_stride, table, table_stride, row_slot, row_pos, rows, Hq, Hkv, d, dv, hd, rot, norm,
+                            eps, page_size, has_kv, temp_coef, temp_every, v0, v0_stride, blend, nullptr, nullptr,
+                            nullptr, 1, 0, stream);
 }
 
 LLM_EXPORT int llm_qkv_store(const float* q, int q_stride, const float* k, int k_stride, const float* v,

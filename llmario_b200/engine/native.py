@@ -37,6 +37,8 @@ def describe_block(block, shared_tables: Dict[Tuple, torch.Tensor]) -> Optional[
         return None
     if type(block.mixer_norm) is not RmsNorm or type(block.ffn_norm) is not RmsNorm:
         return None
+    if m.general:
+        return None
     if m.position is not None and type(m.position) not in (RotaryHalfSplit, RotaryAdjacentPairs):
         return None         # (adjacent pairs: the mixer has ordered its rows for the kernels' pairs)
     if any(lin.bias is not None for lin in (m.qkv_proj, m.o_proj, f.gate_up, f.down)):
@@ -59,7 +61,7 @@ def describe_block(block, shared_tables: Dict[Tuple, torch.Tensor]) -> Optional[
         p = m.position
         # layers whose rotation has the same constants share one table of angles per step: the
         # driver tells tables apart by the address of the frequencies
-        key = (p.rot_dim, p.theta, p.freq_scale, p.attn_factor, p.inv_freq.device)
+        key = p.constants() + (p.inv_freq.device,)
         table = shared_tables.setdefault(key, p.inv_freq)
         d.rot_dim, d.attn_factor, d.inv_freq = p.rot_dim, p.attn_factor, table.data_ptr()
     else:

@@ -41,6 +41,7 @@ def _signatures():
     return {
         "llm_embed": [P, P, I, P, I, I, I, P, P],
         "llm_rms_norm": [P, P, P, I, P, I, I, F, P],
+        "llm_layer_norm": [P, P, P, P, I, P, I, I, F, P],
         "llm_patch_tokens": [P, P, P, I, P],
         "llm_silu_mul": [P, P, I, I, I, P],
         "llm_add_bias": [P, I, P, I, I, P],
@@ -105,6 +106,8 @@ def _signatures():
         "llm_gated_act": [P, P, P, I, I, I, I, I, P],
         "llm_scale_soft_cap": [P, L, F, F, P],
         "llm_latent_store": [P, I, P, P, P, I, P, P, P, I, L, P, I, P, P, I, I, I, I, I, F, I, I, P],
+        "llm_latent_prepare": [P, I, I, I, P, P, I, P, P, P, P, I, L, P, I, P, P, I, I, I, I, I, I, F, I,
+                               I, P],
         "llm_latent_query": [P, I, P, I, P, P, I, I, I, I, I, I, I, P],
         "llm_gemm_simt_batched": [P, P, P, I, I, I, I, I, I, I, I, I, L, L, L, P],
         "llm_moe_route": [P, I, I, I, I, I, P, P, P, P],
@@ -123,6 +126,9 @@ def _signatures():
         "llm_embed_scaled": [P, P, I, P, I, I, I, P, F, P],
         "llm_qkv_store_mix": [P, I, P, I, P, I, P, P, P, P, P, P, I, L, P, I, P, P, I, I, I, I, I,
                               I, I, I, F, I, I, F, I, P, I, F, P],
+        "llm_qkv_store_maps": [P, I, P, I, P, I, P, P, P, P, P, P, I, L, P, I, P, P, I, I, I, I, I,
+                               I, I, I, F, I, I, F, I, P, I, F, P, P, P, I, I, P],
+        "llm_two_map_heads": [P, P, I, I, I, I, I, F, F, F, P],
         "llm_channel_gate": [P, I, P, I, I, I, I, P],
         "llm_delta_recurrence": [P, I, P, I, P, I, P, I, P, I, P, P, F, I, F, P, L, P, I, P, P, I,
                                  I, I, I, I, I, I, I, P],
@@ -131,6 +137,8 @@ def _signatures():
         "llm_rate_decay": [P, P, P, I, I, I, P],
         "llm_moe_router_scaled": [P, I, P, P, P, I, I, I, I, I, I, I, P, P, P, F, P],
         "llm_moe_route_scaled": [P, I, I, I, I, I, P, P, P, F, P],
+        "llm_moe_router_groups": [P, I, P, P, P, I, I, I, I, I, I, I, P, P, P, F, I, I, P],
+        "llm_moe_route_groups": [P, I, I, I, I, I, P, P, P, F, I, I, P],
     }
 
 
@@ -216,6 +224,20 @@ def rms_norm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: floa
     assert x.shape[1] == width and weight.numel() == width
     _check(lib().llm_rms_norm(_ptr(x), _ptr(weight), _ptr(out), _dt(out), _ptr(rows_index), rows,
                               width, float(eps), _stream()), "rms_norm")
+
+
+def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, out: torch.Tensor,
+               eps: float, rows_index: Optional[torch.Tensor] = None) -> None:
+    """out[r] = d * rsqrt(mean(d^2) + eps) * weight + bias with d = v - mean(v), v =
+    x[rows_index[r] or r]; x, weight, bias float32."""
+    _cuda(x, weight, bias, out, rows_index)
+    assert x.dtype == weight.dtype == bias.dtype == torch.float32
+    assert x.is_contiguous() and out.is_contiguous()
+    rows, width = out.shape
+    assert x.shape[1] == width and weight.numel() == width and bias.numel() == width
+    _check(lib().llm_layer_norm(_ptr(x), _ptr(weight), _ptr(bias), _ptr(out), _dt(out),
+                                _ptr(rows_index), rows, width, float(eps), _stream()),
+           "layer_norm")
 
 
 def silu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> None:
@@ -658,7 +680,9 @@ def qkv_store(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Tens
               norm: int, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor],
               eps: float, rot_dim: int = 0, cos_sin: Optional[torch.Tensor] = None,
               q_temp: Optional[Tuple[float, int]] = None,
-              blend: Optional[Tuple[torch.Tensor, float]] = None) -> None:
+              blend: Optional[Tuple[torch.Tensor, float]] = None, maps: int = 1,
+              biases: Tuple[Optional[torch.Tensor], ...] = (None, None, None),
+              clear: bool = False) -> None:
     """Norm, rotation and stores for the rows of a step.  q float32 [rows, heads * key_dim],
     k [rows, kv_heads * key_dim], v [rows, kv_heads * value_dim] (column slices are fine; k and
     v None: only the queries).  ``norm``: NORM_NONE, NORM_PER_HEAD (weights [key_dim], shared by
@@ -668,7 +692,13 @@ def qkv_store(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Tens
     pages of ``view``; ``head_dim`` >= both sizes is the cache's row, padded with zeros.
     ``q_temp = (coef, every)``: the queries of position p are multiplied by
     ``1 + coef ln(floor((p + 1) / every) + 1)``.  ``blend = (v0, lam)``: what is stored as the
-    value is ``(1 - lam) v + lam v0`` with v0 float32 of v's shape (a column slice is fine)."""
+    value is ``(1 - lam) v + lam v0`` with v0 float32 of v's shape (a column slice is fine).
+    ``biases``: float32 offsets of q, k and v (each optional), added as they are read.  ``maps``: a
+    head has so many queries and keys of ``key_dim`` channels (q [rows, heads * maps * key_dim], k
+    alike, map after map inside a head; norm and rotation per map).  The maps' keys of a head stand
+    side by side in its cache row (``head_dim`` >= maps * key_dim) and every map's query is a row of
+    ``q_out`` [rows, heads * maps * head_dim] of its own that is zero outside its map's channels.
+    ``clear``: what was read of q, k and v is zeroed."""
     _cuda(q, k, v, q_out, q_weight, k_weight, cos_sin, row_slot, row_pos)
     coef, every = q_temp if q_temp is not None else (0.0, 0)
     v0, lam = blend if blend is not None and k is not None else (None, 0.0)
@@ -679,7 +709,11 @@ def qkv_store(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Tens
     has_kv = k is not None
     for t in (q, k, v):
         assert t is None or (t.dtype == torch.float32 and t.stride(1) == 1)
-    assert q_out.is_contiguous() and q_out.shape == (rows, num_heads * head_dim)
+    assert q_out.is_contiguous() and q_out.shape == (rows, num_heads * maps * head_dim)
+    for t, b in ((q, biases[0]), (k, biases[1]), (v, biases[2])):
+        _cuda(b)
+        assert b is None or t is None or (b.dtype == torch.float32 and b.is_contiguous()
+                                          and b.numel() == t.shape[1])
     assert not has_kv or view.k.dtype == q_out.dtype
     if rot_dim:
         assert cos_sin is not None and cos_sin.dtype == torch.float32 and cos_sin.is_contiguous()
@@ -688,14 +722,29 @@ def qkv_store(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Tens
         if norm != NORM_NONE and w is not None:
             assert w.dtype == torch.float32 and w.is_contiguous()
             assert w.numel() == (key_dim if norm == NORM_PER_HEAD else n * key_dim)
-    _check(lib().llm_qkv_store_mix(
+    _check(lib().llm_qkv_store_maps(
         _ptr(q), q.stride(0), _ptr(k), k.stride(0) if has_kv else 0, _ptr(v),
         v.stride(0) if has_kv else 0, _ptr(q_weight), _ptr(k_weight), _ptr(cos_sin), _ptr(q_out),
         _ptr(view.k) if has_kv else None, _ptr(view.v) if has_kv else None, _dt(q_out),
         view.page_stride, _ptr(view.block_table), view.block_table.stride(0), _ptr(row_slot),
         _ptr(row_pos), rows, num_heads, num_kv_heads, key_dim, value_dim, head_dim, rot_dim, norm,
         float(eps), view.page_size, int(has_kv), float(coef), int(every), _ptr(v0),
-        v0.stride(0) if v0 is not None else 0, float(lam), _stream()), "qkv_store")
+        v0.stride(0) if v0 is not None else 0, float(lam), _ptr(biases[0]), _ptr(biases[1]),
+        _ptr(biases[2]), int(maps), int(clear), _stream()), "qkv_store")
+
+
+def two_map_heads(a: torch.Tensor, out: torch.Tensor, heads: int, value_dim: int, weight: float,
+                  diff: float, eps: float) -> None:
+    """out[r, h] = (1 - diff) unit(a[r, h, 0] - weight a[r, h, 1]), unit(.) dividing by the root
+    mean square over the ``value_dim`` channels (eps inside the root), in 32-bit.  a
+    [rows, heads * 2 * n] with n >= value_dim channels per map, out [rows, heads * value_dim]."""
+    _cuda(a, out)
+    rows = a.shape[0]
+    assert a.is_contiguous() and out.is_contiguous() and a.dtype == out.dtype
+    assert a.shape[1] % (2 * heads) == 0 and out.shape == (rows, heads * value_dim)
+    _check(lib().llm_two_map_heads(_ptr(a), _ptr(out), _dt(a), rows, heads, value_dim,
+                                   a.shape[1] // (2 * heads), float(weight), float(diff),
+                                   float(eps), _stream()), "two_map_heads")
 
 
 def pool_blocks(view, pooled_view, row_slot: torch.Tensor, row_pos: torch.Tensor, rows: int,
@@ -1438,6 +1487,31 @@ def latent_query(q: torch.Tensor, cos_sin: Optional[torch.Tensor], q_plain: torc
                                   int(clear), _stream()), "latent_query")
 
 
+def latent_prepare(proj: torch.Tensor, q_col: int, c_col: int, c_weight: torch.Tensor,
+                   cos_sin: Optional[torch.Tensor], q_plain: torch.Tensor, q_full: torch.Tensor,
+                   view, row_slot: torch.Tensor, row_pos: torch.Tensor, heads: int, dim: int,
+                   rot_dim: int, kv_rank: int, eps: float, write_cache: bool = True,
+                   clear: bool = False) -> None:
+    """:func:`latent_query` and the key row of :func:`latent_store` in one launch, for queries
+    that are projected from the mixer's input itself: the columns of proj (float32) from ``q_col``
+    on are the heads' queries, those from ``c_col`` on [latent | key part to rotate]."""
+    _cuda(proj, c_weight, cos_sin, q_plain, q_full, view.k, view.v, row_slot, row_pos)
+    rows = q_plain.shape[0]
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1
+    assert proj.shape[1] >= max(q_col + heads * (dim + rot_dim), c_col + kv_rank + rot_dim)
+    assert q_plain.is_contiguous() and q_full.is_contiguous() and q_plain.dtype == q_full.dtype
+    assert q_plain.dtype == view.k.dtype and c_weight.numel() == kv_rank
+    assert q_full.shape == (rows, heads * (kv_rank + rot_dim)) and q_plain.shape[1] == heads * dim
+    half = 0 if cos_sin is None else cos_sin.shape[1]
+    _check(lib().llm_latent_prepare(
+        _ptr(proj), proj.stride(0), q_col, c_col, _ptr(c_weight), _ptr(cos_sin), half,
+        _ptr(q_plain), _ptr(q_full), _ptr(view.k),
+        _ptr(view.v) if view.v.data_ptr() != view.k.data_ptr() else None, _dt(q_full),
+        view.page_stride, _ptr(view.block_table), view.block_table.stride(0), _ptr(row_slot),
+        _ptr(row_pos), rows, view.page_size, heads, dim, rot_dim, kv_rank, float(eps),
+        int(write_cache), int(clear), _stream()), "latent_prepare")
+
+
 def attention_latent_ok(dtype: torch.dtype, key_dim: int, value_dim: int, page_size: int) -> bool:
     """Whether the tensor-core kernel for attention over latents takes these sizes: bfloat16, key
     rows of whole 16-byte units that fit a CTA's shared memory (up to about 700 channels), pages
@@ -1486,35 +1560,48 @@ def _route_mode(scores: str, correction: Optional[torch.Tensor], experts: int) -
     return ROUTE_MODES[scores]
 
 
+def _group_args(groups: Optional[Tuple[int, int]], experts: int) -> Tuple[int, int]:
+    """(experts of a group, groups kept) as the kernels take them; all groups kept is no choice."""
+    if groups is None:
+        return 0, 0
+    count, keep = groups
+    if count < 1 or experts % count or not 1 <= keep <= count:
+        raise KernelError(f"{keep} of {count} groups of {experts} experts")
+    return (0, 0) if keep == count else (experts // count, keep)
+
+
 def moe_route(z: torch.Tensor, experts: int, top: int, ids: torch.Tensor, wts: torch.Tensor,
               scores: str = "softmax_chosen", correction: Optional[torch.Tensor] = None,
-              weight_scale: float = 1.0) -> None:
+              weight_scale: float = 1.0, groups: Optional[Tuple[int, int]] = None) -> None:
     """Per row the ``top`` largest of the first ``experts`` logits of z (float32, a column slice
     is fine) into ``ids`` (int32 [rows, top]) and the softmax over the chosen into ``wts``.
     ``scores="softmax_all"``: the scores are the softmax over all ``experts`` logits, the choice
     goes by score + ``correction`` (float32 [experts], optional), and a chosen expert's weight is
     its score, not renormalised.  ``"softmax_all_renormed"``: the same choice; the weights are the
     chosen scores over their sum (+ 1e-20), times ``weight_scale``.  ``"sigmoid"``: the largest
-    logits; the weight of a chosen expert is the sigmoid of its logit."""
+    logits; the weight of a chosen expert is the sigmoid of its logit.  ``groups = (count, keep)``:
+    the experts form ``count`` equal groups of neighbours, of which only the ``keep`` with the
+    largest members take part in the choice."""
     _cuda(z, ids, wts, correction)
     mode = _route_mode(scores, correction, experts)
     rows = z.shape[0]
     assert z.dtype == torch.float32 and z.stride(1) == 1 and z.shape[1] >= experts
     assert ids.dtype == torch.int32 and ids.is_contiguous() and ids.shape == (rows, top)
     assert wts.dtype == torch.float32 and wts.is_contiguous() and wts.shape == (rows, top)
-    _check(lib().llm_moe_route_scaled(_ptr(z), z.stride(0), rows, experts, top, mode,
+    size, keep = _group_args(groups, experts)
+    _check(lib().llm_moe_route_groups(_ptr(z), z.stride(0), rows, experts, top, mode,
                                       _ptr(correction), _ptr(ids), _ptr(wts),
-                                      float(weight_scale), _stream()), "moe_route")
+                                      float(weight_scale), size, keep, _stream()), "moe_route")
 
 
 def moe_router(h: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], experts: int,
                top: int, z: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor,
                scores: str = "softmax_chosen", correction: Optional[torch.Tensor] = None,
-               weight_scale: float = 1.0) -> None:
+               weight_scale: float = 1.0, groups: Optional[Tuple[int, int]] = None) -> None:
     """Router logits ``z = h w^T + bias`` (w float32 [n_out, width], sums in 32-bit) and, over
     the first ``experts`` of them, the ``top`` largest per row into ``ids`` with the softmax over
     the chosen into ``wts``: the product and :func:`moe_route` in one launch (``scores``,
-    ``correction`` and ``weight_scale`` as there)."""
+    ``correction``, ``weight_scale`` and ``groups`` as there)."""
     _cuda(h, w, bias, z, ids, wts, correction)
     mode = _route_mode(scores, correction, experts)
     rows, width = h.shape
@@ -1524,10 +1611,11 @@ def moe_router(h: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], e
     assert z.stride(1) == 1 and (bias is None or (bias.dtype == torch.float32 and bias.numel() == n_out))
     assert ids.dtype == torch.int32 and ids.is_contiguous() and ids.shape == (rows, top)
     assert wts.dtype == torch.float32 and wts.is_contiguous() and wts.shape == (rows, top)
-    _check(lib().llm_moe_router_scaled(_ptr(h), _dt(h), _ptr(w), _ptr(bias), _ptr(z),
+    size, keep = _group_args(groups, experts)
+    _check(lib().llm_moe_router_groups(_ptr(h), _dt(h), _ptr(w), _ptr(bias), _ptr(z),
                                        z.stride(0), rows, width, experts, n_out, top, mode,
                                        _ptr(correction), _ptr(ids), _ptr(wts),
-                                       float(weight_scale), _stream()),
+                                       float(weight_scale), size, keep, _stream()),
            "moe_router")
 
 

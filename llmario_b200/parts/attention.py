@@ -33,6 +33,15 @@ Options that are data of the part's spec (each absent by default):
 * tensor role ``gate`` of shape [heads * value_dim, hidden]: a sigmoid gate per output channel
   in the place of one per head.
 
+* ``two_maps = {"diff": c}`` with the tensor roles ``lq1``, ``lk1``, ``lq2``, ``lk2`` ([head_dim] each):
+  every head has two queries and two keys of ``head_dim`` channels (the q and k projections have
+  twice the rows, map after map inside a head; norm and rotation per map) over one value.  With a1
+  and a2 the outputs of the two softmaxes and ``w = exp(lq1 . lk1) - exp(lq2 . lk2) + c`` the head's
+  output is ``(1 - c) unit(a1 - w a2)``, unit(.) dividing by the root mean square over the head's
+  channels (``eps``).  In the cache the two keys of a head share one row [key 1 | key 2] beside the
+  value; a map's query is a row of its own, zero where the other map's key stands, so a step reads
+  every key and value once for both maps.  Takes a chunked mask.
+
 These run through the store kernel of ``csrc/qkv_store.cu`` (which also turns adjacent
 pairs itself; the pairs (i, i + rot_dim/2) of ``rope_neox`` are brought side by side by
 ordering the rows of the q and k projections accordingly) and the attention call with the
@@ -97,7 +106,13 @@ class Attention:
         self.gate_per_channel = gate_entry is not None and \
             int(gate_entry[1][0]) == self.num_heads * self.value_dim != self.num_heads
         # what the store kernel of several forms serves (see the module's text)
-        self.general = bool(self.keep_first or self.sink is not None or self.shared_kv
+        self.maps, self.diff = 1, 0.0
+        if spec.get("two_maps") is not None:
+            self.maps, self.diff, self.eps = 2, float(spec["two_maps"]["diff"]), float(spec["eps"])
+            lam = [tensor_of(spec, r, weights).to(torch.float32) for r in ("lq1", "lk1", "lq2", "lk2")]
+            self.second_weight = float(torch.exp((lam[0] * lam[1]).sum())
+                                       - torch.exp((lam[2] * lam[3]).sum())) + self.diff
+        self.general = bool(self.maps > 1 or self.keep_first or self.sink is not None or self.shared_kv
                             or self.value_dim != self.head_dim or self.q_temp is not None
                             or self.blend_group is not None or self.gate_per_channel)
         if self.general:
@@ -164,15 +179,27 @@ class Attention:
         self.o_proj = Linear(tensor_of(spec, "o", weights), b["o"])
 
     def _init_general(self, spec: PartSpec, weights, dtype, device) -> None:
-        if self.chunk is not None or self.values_are_keys:
+        if self.maps > 1 and (self.keep_first or self.shared_kv or self.blend_group is not None
+                              or spec["tensors"].get("gate") is not None or self.sink is not None):
+            raise ConfigError("attention: two maps do not combine with kept first keys, a sink, "
+                              "shared keys and values, blended values or a gate")
+        if (self.chunk is not None and self.maps == 1) or self.values_are_keys:
             raise ConfigError("attention: kept first keys, a sink, shared keys and values, a "
                               "value size of its own, a query temperature or blended values do "
                               "not combine with a chunked mask or values that are keys")
         if self.blend_group is not None and self.shared_kv:
             raise ConfigError("attention: a layer without values of its own blends none")
         d, dv = self.head_dim, self.value_dim
-        self.cache_dim = max(d, dv)
-        refusal = kernels.attention_refusal(self.num_heads, self.num_kv_heads, self.cache_dim)
+        self.cache_dim = max(self.maps * d, dv)
+        if self.maps > 1:
+            # a little padding brings the row to a size the tensor-core kernels have
+            for size in (64, 128):
+                if self.cache_dim <= size < 1.4 * self.cache_dim and dtype == torch.bfloat16 and \
+                        128 % (self.maps * self.num_heads // self.num_kv_heads) == 0:
+                    self.cache_dim = size
+                    break
+        refusal = kernels.attention_refusal(self.maps * self.num_heads, self.num_kv_heads,
+                                            self.cache_dim)
         if refusal is not None:
             raise ConfigError(f"attention: {refusal}")
         self.position = (build_part("position", spec["position"], weights, dtype, device)
@@ -185,8 +212,8 @@ class Attention:
             raise ValueError("q_norm and k_norm must share eps")
         if (self.q_norm is None) != (self.k_norm is None) and not self.shared_kv:
             raise ValueError("q_norm and k_norm come together")
-        self.q_width = self.num_heads * d
-        self.k_cols, self.v_cols = self.num_kv_heads * d, self.num_kv_heads * dv
+        self.q_width = self.num_heads * self.maps * d
+        self.k_cols, self.v_cols = self.num_kv_heads * self.maps * d, self.num_kv_heads * dv
         roles = ["q"] + ([] if self.shared_kv else ["k", "v"])
         w = {r: tensor_of(spec, r, weights) for r in roles}
         b = {r: optional_tensor_of(spec, r + "_bias", weights) for r in roles + ["o"]}
@@ -198,7 +225,7 @@ class Attention:
             _, rot, _ = self.position.rotary_tables()
             order = [j for i in range(rot // 2) for j in (i, i + rot // 2)] + list(range(rot, d))
             perm = torch.tensor(order, dtype=torch.long, device=w["q"].device)
-            for r, heads in (("q", self.num_heads), ("k", self.num_kv_heads)):
+            for r, heads in (("q", self.num_heads * self.maps), ("k", self.num_kv_heads * self.maps)):
                 if r not in w:
                     continue
                 w[r] = w[r].view(heads, d, -1)[:, perm].reshape(w[r].shape)
@@ -229,6 +256,12 @@ class Attention:
             mats.append(torch.zeros(16 - n_rows % 16, self.hidden, dtype=mats[0].dtype,
                                     device=mats[0].device))
             biases.append(None)
+        self.qkv_biases = (None, None, None)
+        if self.maps > 1:       # the store kernel adds the biases as it reads
+            self.qkv_biases = tuple(None if b[r] is None else
+                                    b[r].to(device=device, dtype=torch.float32).contiguous()
+                                    for r in ("q", "k", "v"))
+            biases = None
         self.qkv_proj = Linear.stacked(mats, biases)
         # (attention writes value_dim channels per head, so the projection is as stored)
         self.o_proj = Linear(tensor_of(spec, "o", weights), b["o"])
@@ -256,7 +289,7 @@ class Attention:
     def cache_need(self):
         # (no query ever looks back further than a chunk is long: pages behind that go back)
         if self.general:
-            return PagedKV(self.num_kv_heads, self.cache_dim, self.cache_window,
+            return PagedKV(self.num_kv_heads, self.cache_dim, self.cache_window or self.chunk,
                            self.cache_keep_first if self.cache_window else 0)
         return PagedKV(self.num_kv_heads, self.head_dim, self.window or self.chunk)
 
@@ -272,6 +305,46 @@ class Attention:
         proj = ctx.buffer(name, (ctx.rows, self.qkv_proj.out_features), torch.float32)
         self.qkv_proj(h, proj)
         self._run_general(ctx, call, proj, x, accumulate)
+
+    def _forward_maps(self, ctx: StepContext, call: BoundCall, h: torch.Tensor, x: torch.Tensor,
+                      accumulate: bool) -> None:
+        rows, d, dv, hd = ctx.rows, self.head_dim, self.value_dim, self.cache_dim
+        view = ctx.cache.view(call.cache_entry)
+        if view is None:
+            raise RuntimeError(f"run-order entry {call.index}: attention needs a cache")
+        if not call.writes_cache:
+            raise RuntimeError(f"run-order entry {call.index}: attention with two maps keeps a "
+                               "cache of its own")
+        # (few rows: the product adds partial sums into a buffer kept at zero, which the store
+        # kernel clears as it reads)
+        kept_zero = rows <= kernels.SPLIT_K_MAX_ROWS
+        width = self.qkv_proj.out_features
+        proj = ctx.buffer("attn.proj.%s%d" % ("z" if kept_zero else "", width), (rows, width),
+                          torch.float32, zero=kept_zero)
+        self.qkv_proj(h, proj, out_is_zero=kept_zero)
+        cos_sin, rot = None, 0
+        if self.position is not None:
+            _, rot, _ = self.position.rotary_tables()
+            cos_sin = self.position.step_angles(ctx)
+        heads, a = self.maps * self.num_heads, self.q_width + self.k_cols
+        q = ctx.buffer("attn.q", (rows, heads * hd))
+        kernels.qkv_store(
+            proj[:, :self.q_width], proj[:, self.q_width:a], proj[:, a:a + self.v_cols], q, view,
+            ctx.row_slot, ctx.row_pos, self.num_heads, self.num_kv_heads, d, dv, hd,
+            kernels.NORM_PER_HEAD if self.q_norm is not None else kernels.NORM_NONE,
+            self.q_norm.weight if self.q_norm is not None else None,
+            self.k_norm.weight if self.k_norm is not None else None,
+            self.q_norm.eps if self.q_norm is not None else 0.0, rot, cos_sin,
+            q_temp=self.q_temp, maps=self.maps, biases=self.qkv_biases, clear=kept_zero)
+        # the tensor-core kernels write whole rows, the others stop behind the value
+        whole = driver.tensor_core_attention(ctx.dtype, view, heads, self.num_kv_heads, hd)
+        n = hd if whole else dv
+        maps = ctx.buffer("attn.maps", (rows, heads * n))
+        driver.attention(ctx, q, maps, view, heads, self.num_kv_heads, hd, self.scale, self.mask,
+                         value_dim=None if n == hd else n)
+        out = ctx.buffer("attn.out", (rows, self.num_heads * dv))
+        kernels.two_map_heads(maps, out, self.num_heads, dv, self.second_weight, self.diff, self.eps)
+        self.o_proj(out, x, accumulate=accumulate)
 
     def _run_general(self, ctx: StepContext, call: BoundCall, proj: torch.Tensor,
                      x: torch.Tensor, accumulate: bool) -> None:
@@ -327,6 +400,9 @@ class Attention:
     def forward(self, ctx: StepContext, call: BoundCall, h: torch.Tensor, x: torch.Tensor,
                 accumulate: bool = True) -> None:
         """Adds the result into ``x``; with ``accumulate=False`` ``x`` (float32) receives it."""
+        if self.maps > 1:
+            self._forward_maps(ctx, call, h, x, accumulate)
+            return
         if self.general:
             self._forward_general(ctx, call, h, x, accumulate)
             return

@@ -26,6 +26,9 @@ class PreNormResidualBlock:
         self.mixer = build_part("mixer", layer.mixer, weights, dtype, device)
         self.feed_forward = build_part("feed_forward", layer.feed_forward, weights, dtype,
                                        device)
+        # (see HyperConnectionBlock.forward: mixers of several small kernels in front of products of
+        # many rows)
+        self.ordered_rows = int(spec.get("plain_order_rows") or 0)
         if self.ffn_norm is None and layer.feed_forward.kind != "none":
             raise ConfigError("a pre-norm block with a feed-forward needs its norm")
 
@@ -44,6 +47,12 @@ class PreNormResidualBlock:
                                            self.feed_forward) if p is not None)
 
     def forward(self, ctx: StepContext, call: BoundCall, x: torch.Tensor) -> None:
+        order = kernels.plain_stream_order() if 0 < self.ordered_rows <= ctx.rows \
+            else contextlib.nullcontext()
+        with order:
+            self._forward(ctx, call, x)
+
+    def _forward(self, ctx: StepContext, call: BoundCall, x: torch.Tensor) -> None:
         h = ctx.buffer("block.h", x.shape)
         self.mixer_norm.apply(ctx, x, h)
         self.mixer.forward(ctx, call.for_need(0) if call.cache_entries else call, h, x)

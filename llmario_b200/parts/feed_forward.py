@@ -16,6 +16,8 @@ output is the input itself); ``activation: "clamped_swish"`` with ``limit``;
 their sum, times ``weight_scale``); ``activation: "relu_squared"`` (experts without a gate,
 ``W_down max(W_up h, 0)^2``: there are no ``gate<e>`` tensors); ``scores: "sigmoid"`` (the largest
 logits are chosen; a chosen expert's weight is the sigmoid of its logit, not renormalised);
+``groups = {"count": n, "keep": m}`` (the experts form n equal groups of neighbours and only those
+of the m groups with the largest members can be chosen);
 ``weight_on: "input"`` (a chosen expert reads its weight times the token's input, and its output is
 added as it is).
 
@@ -204,6 +206,14 @@ class RoutedExperts:
                               "'softmax_all_renormed'")
         if not 1 <= self.top <= min(self.routed, 16):
             raise ConfigError(f"routed experts: top {self.top} of {self.routed} (at most 16)")
+        self.groups = None
+        if spec.get("groups") is not None:
+            count, keep = int(spec["groups"]["count"]), int(spec["groups"]["keep"])
+            if count < 1 or self.routed % count or not 1 <= keep <= count or \
+                    keep * (self.routed // count) < self.top:
+                raise ConfigError(f"routed experts: top {self.top} out of {keep} of {count} groups "
+                                  f"of {self.routed} experts")
+            self.groups = (count, keep)
         router = tensor_of(spec, "router", weights).to(torch.float32)
         if router.shape[0] != self.routed:
             raise ConfigError(f"routed experts: a router of {router.shape[0]} outputs for "
@@ -267,11 +277,11 @@ class RoutedExperts:
         wts = ctx.buffer("moe.weights", (rows, top), torch.float32)
         if (self.hidden + self.router.out_features) * 4 <= 200 * 1024:
             kernels.moe_router(h, self.router.weight, self.router.bias, R, top, z, ids, wts,
-                               self.scores, self.correction, self.weight_scale)
+                               self.scores, self.correction, self.weight_scale, self.groups)
         else:           # a row too wide to stage: the product, then the choice
             self.router(h, z)
             kernels.moe_route(z, R, top, ids, wts, self.scores, self.correction,
-                              self.weight_scale)
+                              self.weight_scale, self.groups)
         ident = h if self.identity else None
         shared = gate = None
         kept_zero = rows <= kernels.SPLIT_K_MAX_ROWS

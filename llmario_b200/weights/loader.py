@@ -38,12 +38,12 @@ class WeightError(ValueError):
         super().__init__("\n".join(lines))
 
 
-def _walk(part: PartSpec) -> Iterator[Tuple[str, Tuple[int, ...]]]:
+def _walk(part: PartSpec) -> Iterator[Tuple[str, Tuple[int, ...], Optional[float]]]:
+    """(name, shape, mean of random values or None) of every tensor ``part`` lists."""
     for key, value in part.params.items():
         if key == "tensors":
             for entry in value.values():
-                name, shape = entry[0], tuple(entry[1])
-                yield name, shape
+                yield entry[0], tuple(entry[1]), entry[2] if len(entry) > 2 else None
         elif isinstance(value, PartSpec):
             yield from _walk(value)
         elif isinstance(value, (list, tuple)):
@@ -52,14 +52,18 @@ def _walk(part: PartSpec) -> Iterator[Tuple[str, Tuple[int, ...]]]:
                     yield from _walk(v)
 
 
-def expected_tensors(spec: ModelSpec) -> Dict[str, Tuple[int, ...]]:
-    """name -> shape for every tensor the parts of ``spec`` ask for."""
-    out: Dict[str, Tuple[int, ...]] = {}
+def _parts(spec: ModelSpec) -> List[PartSpec]:
     parts = [spec.embedding, spec.final_norm, spec.head]
     for layer in spec.layers:
         parts += [layer.block, layer.mixer, layer.feed_forward]
-    for part in parts:
-        for name, shape in _walk(part):
+    return parts
+
+
+def expected_tensors(spec: ModelSpec) -> Dict[str, Tuple[int, ...]]:
+    """name -> shape for every tensor the parts of ``spec`` ask for."""
+    out: Dict[str, Tuple[int, ...]] = {}
+    for part in _parts(spec):
+        for name, shape, _ in _walk(part):
             if name in out and out[name] != shape:
                 raise WeightError([], [], [(name, shape, out[name])], "the model's own spec")
             out[name] = shape
@@ -126,7 +130,8 @@ def load_weights(model_dir: str, spec: ModelSpec, dtype: torch.dtype,
 def random_tensors(spec: ModelSpec, seed: int, dtype: torch.dtype,
                    device: torch.device | str = "cpu", matrix_std: float = 0.02,
                    gain_std: float = 0.01) -> Dict[str, torch.Tensor]:
-    """Seeded weights: matrices ~ N(0, matrix_std), one-dimensional gains (and single numbers) 1 + N(0, gain_std).
+    """Seeded weights: matrices ~ N(0, matrix_std), one-dimensional gains (and single numbers) 1 + N(0, gain_std);
+    a tensor that is listed as (name, shape, mean) has that mean in place of 0 or 1 (offsets, for instance).
     Every element is a function of (seed, tensor name, element index) alone
     (:mod:`.random_normal`): the values are the same bits on a CUDA device (made by the kernel
     of ``csrc/random_weights.cu``) and on the host (made by NumPy), and do not depend on the
@@ -135,10 +140,12 @@ def random_tensors(spec: ModelSpec, seed: int, dtype: torch.dtype,
 
     out: Dict[str, torch.Tensor] = {}
     device = torch.device(device)
+    means = {name: mean for part in _parts(spec) for name, _, mean in _walk(part)}
     for name, shape in expected_tensors(spec).items():
         key = tensor_key(seed, name)
         shape = tuple(FREE_DIM_DEFAULT if d is None else d for d in shape)
         mean, std = (1.0, gain_std) if len(shape) <= 1 else (0.0, matrix_std)
+        mean = mean if means[name] is None else means[name]
         t = torch.empty(shape, dtype=dtype, device=device)
         if device.type == "cuda":
             from .. import kernels
