@@ -76,10 +76,17 @@ MOMUVIK_PRESETS = {"momuvik-0.6b": ("qwen3-0.6b", 28), "momuvik-8b": ("qwen3-8b"
                    "momuvik-tiny": ("tiny-b", 4)}
 
 
+# Ronurax models of the same sizes (random weights): latent attention three times, then attention
+# with two maps in chunks; routed experts everywhere.
+RONURAX_PRESETS = {"ronurax-0.6b": ("qwen3-0.6b", 28), "ronurax-8b": ("qwen3-8b", 36),
+                   "ronurax-tiny": ("tiny-b", 4)}
+
+
 def is_preset(name: str) -> bool:
     return name.lower() in PRESETS or name.lower() in VUNASUN_PRESETS \
         or name.lower() in RUNIDRA_PRESETS or name.lower() in PEMOLORN_PRESETS \
-        or name.lower() in PAVATAR_PRESETS or name.lower() in MOMUVIK_PRESETS
+        or name.lower() in PAVATAR_PRESETS or name.lower() in MOMUVIK_PRESETS \
+        or name.lower() in RONURAX_PRESETS
 
 
 def preset_config(name: str, num_layers: Optional[int] = None):
@@ -134,6 +141,17 @@ def preset_config(name: str, num_layers: Optional[int] = None):
         return momuvik_sized_like(p["hidden_size"], p["intermediate_size"],
                                   p["num_attention_heads"], int(num_layers or layers),
                                   p["vocab_size"], **small)
+
+    if name.lower() in RONURAX_PRESETS:
+        from .config.ronurax import sized_like as ronurax_sized_like
+
+        base, layers = RONURAX_PRESETS[name.lower()]
+        p = PRESETS[base]
+        small = {"kv_rank": 56, "rot": 16, "chunk": 24} if base.startswith("tiny") else {}
+        return ronurax_sized_like(p["hidden_size"], p["intermediate_size"],
+                                  p["num_attention_heads"], p["num_key_value_heads"],
+                                  p["head_dim"], int(num_layers or layers), p["vocab_size"],
+                                  **small)
 
     raw = dict(PRESETS[name.lower()], architectures=["Qwen3ForCausalLM"], model_type="qwen3")
     if num_layers:
@@ -308,7 +326,7 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
     sub = ap.add_subparsers(dest="cmd", required=True)
     run = sub.add_parser("run", help="generate from a prompt of token ids")
     run.add_argument("model", help="model folder, or a preset name: " + ", ".join(list(PRESETS) + list(VUNASUN_PRESETS) + list(RUNIDRA_PRESETS) + list(PEMOLORN_PRESETS) + list(PAVATAR_PRESETS)
-                     + list(MOMUVIK_PRESETS)))
+                     + list(MOMUVIK_PRESETS) + list(RONURAX_PRESETS)))
     run.add_argument("--tokens", default=None, help="comma-separated prompt token ids")
     run.add_argument("--prompt-len", type=int, default=16,
                      help="without --tokens: this many random ids")

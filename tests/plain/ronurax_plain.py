@@ -186,19 +186,20 @@ def choose(scores, top: int, count: int, keep: int):
 
 def choice_margin(z, top: int, count: int, keep: int):
     """Per row of router outputs, by how much they would have to change for another choice: the
-    distance of the last kept group to the first one left out, and of the last chosen expert to
-    the best one left out in the kept groups."""
+    distance of the last chosen expert to the best one left out in the kept groups and, when the
+    last kept group holds a chosen expert, of that group to the first one left out."""
     T, E = z.shape
     size = E // count
     best = z.reshape(T, count, size).max(axis=2)
+    ids = choose(z, top, count, keep)
     least = np.full(T, np.inf)
     for i in range(T):
         order = np.argsort(-best[i], kind="stable")
-        if keep < count:
+        if keep < count and (ids[i] // size == order[keep - 1]).any():
             least[i] = best[i, order[keep - 1]] - best[i, order[keep]]
-        inside = sorted((z[i, e] for e in range(E) if e // size in order[:keep]), reverse=True)
-        if top < len(inside):
-            least[i] = min(least[i], inside[top - 1] - inside[top])
+        left = [z[i, e] for e in range(E) if e // size in order[:keep] and e not in ids[i]]
+        if left:
+            least[i] = min(least[i], z[i, ids[i, -1]] - max(left))
     return least
 
 
