@@ -570,12 +570,46 @@ __global__ void channel_gate_kernel(T* __restrict__ out, float* __restrict__ gat
   }
 }
 
+// The same eight bfloat16 channels at a time: cols a multiple of eight, 16-byte aligned rows.
+__global__ void __launch_bounds__(256) channel_gate_vec_kernel(bf16* __restrict__ out, float* __restrict__ gate,
+                                                               int gate_stride, unsigned per_row, unsigned pieces,
+                                                               int clear) {
+  pdl_trigger();
+  pdl_wait();
+  for (unsigned i = blockIdx.x * blockDim.x + threadIdx.x; i < pieces; i += gridDim.x * blockDim.x) {
+    const unsigned r = i / per_row;
+    float4* gp = reinterpret_cast<float4*>(gate + (size_t)r * gate_stride + (i - r * per_row) * 8);
+    uint4* op = reinterpret_cast<uint4*>(out) + i;
+    const float4 a = gp[0], b = gp[1];
+    const uint4 o = *op;
+    if (clear) gp[0] = gp[1] = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float z[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+    const uint32_t u[4] = {o.x, o.y, o.z, o.w};
+    uint32_t w[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const __nv_bfloat162 t =
+          __floats2bfloat162_rn(__uint_as_float(u[j] << 16) / (1.f + expf(-z[2 * j])),
+                                __uint_as_float(u[j] & 0xffff0000u) / (1.f + expf(-z[2 * j + 1])));
+      w[j] = *reinterpret_cast<const uint32_t*>(&t);
+    }
+    *op = make_uint4(w[0], w[1], w[2], w[3]);
+  }
+}
+
 LLM_EXPORT int llm_channel_gate(void* out, int dtype, float* gate, int gate_stride, int rows, int cols, int clear,
                                 cudaStream_t stream) {
   const long long total = (long long)rows * cols;
   if (total <= 0) return 0;
   const int blocks = (int)((total + 255) / 256 < 4736 ? (total + 255) / 256 : 4736);
   // (it stands in front of the output projection: see launched_many_blocks)
+  if (dtype == LLM_BF16 && cols % 8 == 0 && gate_stride % 4 == 0 && (((uintptr_t)out | (uintptr_t)gate) & 15) == 0 &&
+      total < (1LL << 34)) {
+    const unsigned pieces = (unsigned)(total / 8);
+    const int vblocks = (int)((pieces + 255) / 256 < 4736 ? (pieces + 255) / 256 : 4736);
+    return launched_many_blocks(launch_pdl(channel_gate_vec_kernel, vblocks, 256, 0, stream, (bf16*)out, gate,
+                                           gate_stride, (unsigned)cols / 8, pieces, clear), vblocks);
+  }
   if (dtype == LLM_F32)
     return launched_many_blocks(launch_pdl(channel_gate_kernel<float>, blocks, 256, 0, stream, (float*)out, gate,
                                            gate_stride, cols, total, clear), blocks);
