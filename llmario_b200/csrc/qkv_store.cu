@@ -51,11 +51,12 @@ __device__ __forceinline__ void store2(bf16* dst, float a, float b) {
   *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(a, b);
 }
 
+// PIECES: pairs of a head's channels that a lane keeps (with PAIRS, keys of up to 64 * PIECES channels).
 // One block per (row, share of the heads); a warp per head in turn.  With a norm over whole rows
 // every block of a row sums the squares of the whole row itself.  PAIRS: all sizes are even and
-// the rows 8-byte aligned, so a lane reads and writes two adjacent channels at once, which are
-// also the two members of a rotated pair.
-template <typename T, bool PAIRS>
+// the rows 8-byte aligned and a key is not too long, so a lane reads and writes two adjacent channels at
+// once, which are also the two members of a rotated pair.
+template <typename T, bool PAIRS, int PIECES>
 __global__ void __launch_bounds__(256) qkv_store_kernel(const StoreArgs a) {
   __shared__ float scratch[33];
   pdl_trigger();
@@ -127,15 +128,6 @@ __global__ void __launch_bounds__(256) qkv_store_kernel(const StoreArgs a) {
     const float* bias = is_q ? a.q_b : a.k_b;
     if (bias) bias += (size_t)h * a.d;
     float scale = is_q ? whole_q : whole_k;
-    if (a.norm == 1) {
-      float s = 0.f;
-      for (int c = lane; c < a.d; c += 32) {
-        const float x = src[c] + (bias ? bias[c] : 0.f);
-        s = fmaf(x, x, s);
-      }
-      scale = 1.f / sqrtf(warp_sum(s) / (float)a.d + a.eps);
-    }
-    if (is_q) scale *= temp;
     if (w && a.norm == 2) w += (size_t)h * a.d;
     if (!a.norm) w = nullptr;
     // the map's channels start at m * d of its row; a query fills its row, a key what is its own (the
@@ -145,25 +137,48 @@ __global__ void __launch_bounds__(256) qkv_store_kernel(const StoreArgs a) {
              m * a.d;
     const int c0 = is_q ? -m * a.d : 0, c1 = is_q || m == a.maps - 1 ? a.hd - m * a.d : a.d;
     if (PAIRS) {
-      for (int c = c0 + 2 * lane; c < c1; c += 64) {
-        float x = 0.f, y = 0.f;
-        if (c >= 0 && c < a.d) {
-          float2 u = *reinterpret_cast<const float2*>(src + c);
-          if (bias) u.x += bias[c], u.y += bias[c + 1];
-          if (a.clear) *reinterpret_cast<float2*>(const_cast<float*>(src) + c) = make_float2(0.f, 0.f);
-          x = u.x * scale * (w ? w[c] : 1.f);
-          y = u.y * scale * (w ? w[c + 1] : 1.f);
-          if (cs && c < a.rot) {
-            const float2 t = *reinterpret_cast<const float2*>(cs + c);      // (cos, sin) of pair c / 2
-            const float x2 = fmaf(x, t.x, -(y * t.y));
-            y = fmaf(y, t.x, x * t.y);
-            x = x2;
-          }
-        }
-        store2(dst + c, x, y);
+      // everything the head needs is asked for at once and kept in registers
+      float2 u[PIECES], b[PIECES], t[PIECES], g[PIECES];
+      float s = 0.f;
+#pragma unroll
+      for (int i = 0; i < PIECES; ++i) {
+        const int c = 2 * lane + 64 * i;
+        const bool in = c < a.d;
+        u[i] = in ? *reinterpret_cast<const float2*>(src + c) : make_float2(0.f, 0.f);
+        b[i] = in && bias ? *reinterpret_cast<const float2*>(bias + c) : make_float2(0.f, 0.f);
+        t[i] = cs && c < a.rot ? *reinterpret_cast<const float2*>(cs + c) : make_float2(1.f, 0.f);   // (cos, sin) of pair c / 2
+        g[i] = in && w ? *reinterpret_cast<const float2*>(w + c) : make_float2(1.f, 1.f);
       }
+#pragma unroll
+      for (int i = 0; i < PIECES; ++i) {
+        u[i].x += b[i].x, u[i].y += b[i].y;
+        s = fmaf(u[i].x, u[i].x, s), s = fmaf(u[i].y, u[i].y, s);
+      }
+      if (a.norm == 1) scale = 1.f / sqrtf(warp_sum(s) / (float)a.d + a.eps);
+      if (is_q) scale *= temp;
+#pragma unroll
+      for (int i = 0; i < PIECES; ++i) {
+        const int c = 2 * lane + 64 * i;
+        if (c < a.d) {
+          const float x = u[i].x * scale * g[i].x, y = u[i].y * scale * g[i].y;
+          store2(dst + c, fmaf(x, t[i].x, -(y * t[i].y)), fmaf(y, t[i].x, x * t[i].y));
+        }
+      }
+      if (a.clear)
+        for (int c = 2 * lane; c < a.d; c += 64) *reinterpret_cast<float2*>(const_cast<float*>(src) + c) = make_float2(0.f, 0.f);
+      for (int c = c0 + 2 * lane; c < 0; c += 64) store2(dst + c, 0.f, 0.f);
+      for (int c = a.d + 2 * lane; c < c1; c += 64) store2(dst + c, 0.f, 0.f);
       continue;
     }
+    if (a.norm == 1) {
+      float s = 0.f;
+      for (int c = lane; c < a.d; c += 32) {
+        const float x = src[c] + (bias ? bias[c] : 0.f);
+        s = fmaf(x, x, s);
+      }
+      scale = 1.f / sqrtf(warp_sum(s) / (float)a.d + a.eps);
+    }
+    if (is_q) scale *= temp;
     for (int c = c0 + lane; c < c1; c += 32) {
       float x = 0.f;
       if (c >= 0 && c < a.d) {
@@ -257,20 +272,22 @@ LLM_EXPORT int llm_qkv_store_maps(const float* q, int q_stride, const float* k, 
   const int heads = Hq * maps + (has_kv ? (maps + 1) * Hkv : 0);
   const int threads = heads >= 8 ? 256 : heads >= 4 ? 128 : 64;
   // few rows: the heads of a row are shared out to several blocks, so that the step fills the GPU
-  int shares = 1;
+  int shares = rows < 4096 && norm != 2 ? 2 : 1;
   if (rows < 1024) {
     shares = (heads + threads / 32 - 1) / (threads / 32);
     if (shares > 8) shares = 8;
   }
-  const bool even = !((d | dv | hd | q_stride) & 1) && !((uintptr_t)q & 7) && !((uintptr_t)q_out & 7) &&
+  const bool even = d <= 256 && !(((uintptr_t)q_w | (uintptr_t)k_w | (uintptr_t)q_b | (uintptr_t)k_b) & 7) && !((d | dv | hd | q_stride) & 1) && !((uintptr_t)q & 7) && !((uintptr_t)q_out & 7) &&
                     (!has_kv || (!((k_stride | v_stride) & 1) && !(page_stride & 1) &&
                                  !(((uintptr_t)k | (uintptr_t)v | (uintptr_t)k_cache | (uintptr_t)v_cache) & 7))) &&
                     (rot == 0 || !((uintptr_t)cos_sin & 7));
   const dim3 grid(rows, shares);
   int rc;
 #define STORE_GO(T) \
-  rc = even ? launch_pdl(qkv_store_kernel<T, true>, grid, threads, 0, stream, a) \
-            : launch_pdl(qkv_store_kernel<T, false>, grid, threads, 0, stream, a)
+  rc = !even      ? launch_pdl(qkv_store_kernel<T, false, 1>, grid, threads, 0, stream, a) \
+       : d <= 64  ? launch_pdl(qkv_store_kernel<T, true, 1>, grid, threads, 0, stream, a)  \
+       : d <= 128 ? launch_pdl(qkv_store_kernel<T, true, 2>, grid, threads, 0, stream, a)  \
+                  : launch_pdl(qkv_store_kernel<T, true, 4>, grid, threads, 0, stream, a)
   if (dtype == LLM_F32) STORE_GO(float);
   else if (dtype == LLM_BF16) STORE_GO(bf16);
   else return LLM_ERR_UNSUPPORTED;
