@@ -276,7 +276,7 @@ def sized_like(width: int, ff: int, heads: int, kv_heads: int, head_dim: int, la
               "scale": (head_dim + rot) ** -0.5,
               "rot": {"dims": rot, "base": 1e6, "scaling": {"factor": 4.0, "original": 4096,
                                                             "fast": 32.0, "slow": 1.0}}}
-    maps = {"heads": heads, "kv_heads": kv_heads, "dim": half, "vdim": head_dim, "diff": 0.3,
+    maps = {"heads": heads, "kv_heads": kv_heads, "dim": half, "vdim": head_dim, "diff": 0.35,
             "scale": half ** -0.5, "mask": {"size": chunk},
             "rot": {"dims": half, "base": 5e5, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0,
                                                            "original": 4096}}}

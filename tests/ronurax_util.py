@@ -88,8 +88,8 @@ CONFIGS: Dict[str, dict] = {
     "map_one": config([maps(heads=1, kv=1, dim=8, vdim=12, chunk=5, rot=2, diff=0.8)], width=40),
     # chunks of one position, chunks longer than a prompt, no chunks; no rotation, no scaling
     "chunk_1": config([maps(chunk=1), latent()]),
-    "chunk_long": config([maps(heads=4, kv=2, dim=32, vdim=64, chunk=700, rot=32)]),
-    "chunk_none": config([maps(chunk=0, dim=32, vdim=64), maps(chunk=0, rot=0)]),
+    "chunk_long": config([maps(heads=6, kv=2, dim=32, vdim=64, chunk=700, rot=32)]),
+    "chunk_none": config([maps(heads=3, kv=3, chunk=0, dim=32, vdim=64), maps(chunk=0, rot=0)]),
     "no_scaling": config([maps(scaling=None), latent(scaling=None), latent(rot_dim=0, kv_rank=40)]),
     # key rows of latents for every kernel: 64 and 128 channels (with and without fitting heads),
     # several blocks of 64, values in parts
@@ -154,7 +154,7 @@ def random_config(seed: int) -> str:
             layers.append(latent(heads=pick(2, 4, 5, 8, 12), dim=pick(24, 32, 48), rot_dim=pick(8, 16, 32),
                                  vdim=pick(24, 40, 56), kv_rank=pick(48, 64, 88, 112, 160), mlp=mlp,
                                  base=pick(1e4, 5e5), scale=pick(None, 0.15),
-                                 scaling=pick((3.0, 64, 20.0, 1.5), (2.0, 512, 32.0, 1.0), (6.0, 100, 8.0, 2.0))))
+                                 scaling=pick((3.0, 64, 20.0, 1.5), (2.5, 400, 24.0, 1.0), (6.0, 100, 8.0, 2.0))))
     CONFIGS[name] = config(layers, width=pick(88, 128, 160, 208), vocab=int(rng.integers(150, 500)),
                            eps=pick(1e-6, 1e-5))
     return name

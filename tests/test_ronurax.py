@@ -719,7 +719,7 @@ def test_a_key_that_stands_out_far_back(dtype, page, kv_rank, rot, heads):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("which", (0, 1))
 @pytest.mark.parametrize("page,chunk,dim,vdim,heads,kv", [
-    (16, 50, 32, 64, 4, 2), (64, 96, 64, 128, 8, 2), (16, 41, 20, 28, 4, 1), (32, 32, 24, 40, 2, 2), (64, 200, 16, 64, 8, 1)])
+    (16, 50, 32, 64, 6, 3), (64, 96, 64, 128, 8, 2), (16, 41, 20, 28, 4, 1), (32, 32, 24, 40, 2, 2), (64, 200, 16, 64, 8, 1)])
 def test_a_key_that_stands_out_at_a_chunk_edge(dtype, which, page, chunk, dim, vdim, heads, kv):
     """A needle on the last place of a chunk (no probe of the next chunk sees it) and one on the first
     place (every probe of its chunk does), in a prompt, in portions cut around the edge, and decoded
